@@ -31,7 +31,7 @@
 extern "C" {
 #endif
 
-#define LCC_ABI_VERSION 11
+#define LCC_ABI_VERSION 12
 #define LCC_PAGE_SIZE 64
 
 typedef struct lcc_ctx lcc_ctx;
@@ -297,7 +297,8 @@ int lcc_resize_bicubic_aa_u8(lcc_ctx* ctx, const lcc_resize_plan* plan, const ui
  * or, in a model with LCC_BLOCK_PRENORM_HC, pre-norm sublayers on several residual streams (see LCC_BLOCK_PRENORM_HC),
  * or, with LCC_BLOCK_PARALLEL, x <- x + mixer(norm1(x)) + ff(norm1(x)),
  * or, with LCC_BLOCK_BRANCHNORM, x <- x + norm1(mixer(x + canon(x))), then x <- x + norm2(ff(x)) (the norm sits on the sublayer's
- * output; canon is a short causal convolution over time on every channel of the residual stream);
+ * output; canon is a short causal convolution over time on every channel of the residual stream),
+ * or, with LCC_BLOCK_SANDWICH, x <- x + norm1b(mixer(norm1(x))), then x <- x + norm2b(ff(norm2(x)));
  * the feed-forward is dense (gated gelu, or two matrices around a gelu) or routed (LCC_FF_MOE);
  * with the residual stream(s), every norm, every score, every router and every recurrent state in fp32. One library serves two storage
  * types: LCC_DT_BF16 (bf16 weights, activations and K/V pages; fp32 accumulation) and LCC_DT_F32 (everything fp32, plain
@@ -309,28 +310,34 @@ int lcc_resize_bicubic_aa_u8(lcc_ctx* ctx, const lcc_resize_plan* plan, const ui
 #define LCC_MIX_RETENTION 3 /* rotary q/k -> linear attention with a fixed decay per head, no normaliser -> unit-rms heads x silu gate -> out-proj */
 #define LCC_MIX_LATENT 4    /* causal softmax attention over a cached low-rank latent + one shared rotary key part, per-head sink and sigmoid gate */
 #define LCC_MIX_ATTENTION 5 /* softmax attention over paged K/V: per-head q/k RMS norm, rotary positions on part of a head, a sliding
-                               window and / or chunks, optional sink, values projected or taken from the keys as projected, output
-                               gate per head or per channel (every option a field of the layer) */
+                               window (which may keep the first positions) and / or chunks, optional sink, values projected or taken
+                               from the keys as projected, output gate per head or per channel, soft-capped scores, two maps per head
+                               whose normed difference is the output (every option a field of the layer) */
 #define LCC_MIX_DELTA 6     /* gated delta rule with a decay per key channel: q/k/v through a short causal convolution + silu, unit-length q
                                and k, S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; unit-rms heads x weight x sigmoid
                                gate -> out-proj (decays and output gate come through low-rank bottlenecks) */
 #define LCC_FF_GLU 0        /* dense gated feed-forward: gelu_tanh(gate) * up */
 #define LCC_FF_MOE 1        /* routed experts (sigmoid or softmax router, top-k of score + correction, optionally inside the best groups
                                of neighbouring experts; relu^2 or clamped gated experts; identity experts) + gated shared expert */
-#define LCC_FF_MLP 2        /* dense two-matrix feed-forward: down(gelu_tanh(up x)) */
+#define LCC_FF_MLP 2        /* dense two-matrix feed-forward: down(act(up x)), act LCC_ACT_* */
+#define LCC_ACT_GELU_TANH 0
+#define LCC_ACT_RELU2 1     /* relu(z)^2 */
 #define LCC_BLOCK_POSTNORM 0 /* x <- norm(alpha * x + sublayer(x)) */
 #define LCC_BLOCK_PRENORM_HC 1 /* `streams` residual streams x_s; per sublayer: u = sum_s in[s] x_s; y = sublayer(norm(u));
                                   x_t <- sum_s mix[s][t] x_s + out[t] y. The model's output is the sum of the streams. */
 #define LCC_BLOCK_PARALLEL 2   /* h = norm1(x); x <- x + mixer(h) + ff(h): one norm, both sublayers read it, one fp32 residual sum */
 #define LCC_BLOCK_BRANCHNORM 3 /* x <- x + norm1(mixer(x + canon(x))); x <- x + norm2(ff(x)): sublayers read the residual stream itself */
+#define LCC_BLOCK_SANDWICH 4   /* x <- x + norm1b(mixer(norm1(x))); x <- x + norm2b(ff(norm2(x))): a norm on either side of a sublayer */
 #define LCC_NORM_RMS 0         /* x / sqrt(mean(x^2) + eps) * w */
 #define LCC_NORM_DYT 1         /* tanh(alpha * x) * w + b: no statistics of the row (Dynamic Tanh) */
+#define LCC_NORM_LAYER 2       /* (x - mean) / sqrt(mean squared deviation + eps) * w, no bias */
 #define LCC_ROUTER_SIGMOID 0
 #define LCC_ROUTER_SOFTMAX 1   /* scores = softmax over all router outputs (identity experts included) */
 #define LCC_ROUTER_TOPK_SOFTMAX 2 /* the e_top largest logits are chosen; weights = softmax over the chosen logits only */
 #define LCC_EXPERT_RELU2 0     /* down(relu(up x)^2) */
 #define LCC_EXPERT_CLAMP_GLU 1 /* g = min(gate x, limit), u = clamp(up x, +-limit); down(g * sigmoid(1.702 g) * (u + 1)); e_up rows [gate | up] */
 #define LCC_EXPERT_SILU_GLU 2  /* down(silu(gate x) * (up x)); e_up rows as for LCC_EXPERT_CLAMP_GLU */
+#define LCC_EXPERT_GELU 3      /* down(gelu(up x)), the exact (erf) form */
 #define LCC_GATE_NONE 0
 #define LCC_GATE_HEAD 1        /* one sigmoid gate per (row, head) */
 #define LCC_GATE_CHANNEL 2     /* one sigmoid gate per (row, head, value channel) */
@@ -348,6 +355,10 @@ typedef struct {
     float r_tau;
     /* LCC_MIX_RETENTION: heads x dim key channels (the first t_rot_dims of each head rotated), heads x vdim value channels */
     int32_t t_heads, t_dim, t_vdim, t_rot_dims;
+    /* its options (lightning attention sets all four): t_silu: silu on q, k and v; t_plain_keys: no dim^-1/2 on k; t_whole_norm: one RMS
+     * norm over all heads together with the weight t_norm_f32 [heads*vdim] instead of a unit rms per head; t_gate_sigmoid: the gate
+     * is sigmoid(g) instead of silu(g) */
+    int32_t t_silu, t_plain_keys, t_whole_norm, t_gate_sigmoid;
     /* LCC_MIX_LATENT: per head a_dim unrotated + a_rot_dim rotated query channels, value size a_vdim; the cache holds
      * a_rank latent channels + a_rot_dim rotated key channels per token; a_kv_from >= 0: this layer has no cache of its own
      * and reads that layer's */
@@ -370,23 +381,35 @@ typedef struct {
      * cached values are (1 - m_vmix) * v + m_vmix * the kept values of the same token */
     int32_t m_unit_norm, m_vmix_role;
     float m_vmix;
+    /* m_no_qk_norm: q and k as projected; m_keep_first: positions below it stay visible behind the window; m_softcap > 0: scores become
+     * m_softcap * tanh(score / m_softcap); m_maps = 2 (differential attention, 0 reads as 1): each query and key head is two maps of
+     * m_dim channels, each with a softmax of its own over the same values; the output is a1 - m_lambda * a2, brought to unit rms per head,
+     * times m_diff_scale (m_in rows [q: Hq*2*dim | k: G*2*dim | v], K pages [page][G][page_size][2*dim]) */
+    int32_t m_no_qk_norm, m_keep_first, m_maps;
+    float m_softcap, m_lambda, m_diff_scale;
     /* LCC_MIX_DELTA: d_heads value heads of d_vdim channels over d_kv_heads query/key heads of d_dim channels, d_conv taps, bottleneck
      * ranks of the decay and of the output gate */
     int32_t d_heads, d_kv_heads, d_dim, d_vdim, d_conv, d_rank_a, d_rank_g;
     /* feed-forward: ff_kind LCC_FF_*; MoE: e_experts experts of width e_ff, e_top per token, weights = score * e_scale,
      * shared expert of width e_shared_ff (0 = none) */
+    int32_t ff_act;    /* LCC_FF_MLP: LCC_ACT_* */
     int32_t ff_kind, e_experts, e_top, e_ff, e_shared_ff;
     float e_scale;
     /* e_router_kind LCC_ROUTER_*; the last e_identity router outputs (beyond the e_experts real ones) stand for experts that return
      * their input; e_groups > 0: the router outputs form e_groups equal groups of neighbours and only the e_keep groups with the
      * largest choice score can be chosen; e_act LCC_EXPERT_*, e_limit its clamp */
     int32_t e_router_kind, e_identity, e_groups, e_keep, e_act;
+    int32_t e_group_top;       /* a group scores as the sum of that many of its largest choice scores (0 and 1: the largest) */
+    int32_t e_shared_ungated;  /* the shared expert's output is added as it is (the router has no gate row for it) */
     int32_t e_up_il16; /* LCC_EXPERT_CLAMP_GLU: non-zero when each expert's gate and up rows are interleaved in groups of 16 (16 gate
                           rows, then the 16 matching up rows; e_ff a multiple of 16) instead of [gate: e_ff | up: e_ff] */
     float e_limit;
     float norm1_alpha; /* LCC_NORM_DYT: the scalar inside tanh */
     /* weights: matrices [out, in] in the model's storage type; everything named *_f32 is fp32 */
     const float *norm1_f32, *norm2_f32;
+    const float *norm1b_f32, *norm2b_f32; /* LCC_BLOCK_SANDWICH: the norms behind the sublayers */
+    const float* m_in_bias_f32;  /* biases of the q, k, v rows of m_in (NULL: none) */
+    const void* m_in_bias;       /* optional copy in the storage type, padded like the matrix rows (tensor-core epilogue) */
     const float* canon_w_f32;  /* LCC_BLOCK_BRANCHNORM: [width, canon_taps] taps of the convolution in front of the mixer (NULL: none) */
     const float* m_temp_f32;   /* [m_heads] or NULL */
     const void* a_uq;          /* [heads*(dim+rot_dim), a_q_rank] */
@@ -424,7 +447,7 @@ typedef struct {
     const float* rot_inv_freq_f32; /* [rot dims / 2]: rotation frequencies of this layer's mixer, computed by the host */
     const void* t_in;          /* [2*heads*dim + 2*heads*vdim, width], rows [q | k | v | gate] */
     const float* t_log_decay_f32; /* [heads]: log of the per-head decay */
-    const float* t_norm_f32;   /* [vdim]: weight of the per-head unit norm (ones when the design has none) */
+    const float* t_norm_f32;   /* [vdim]: weight of the per-head unit norm (ones when the design has none); t_whole_norm: [heads*vdim] */
     const void* t_out;         /* [width, heads*vdim] */
     const void* a_in;          /* [heads*(dim+rot_dim) (+ rank + rot_dim) + heads, width], rows [q | latent, key part | gate];
                                   a layer that reads another layer's cache has no middle block */
@@ -449,7 +472,7 @@ typedef struct {
     float eps, alpha, embed_scale, logit_softcap; /* logit_softcap <= 0: none */
     int32_t block;   /* LCC_BLOCK_* */
     int32_t streams; /* residual streams of LCC_BLOCK_PRENORM_HC (>= 1) */
-    int32_t norm_kind; /* LCC_NORM_*: the block norms and the final norm */
+    int32_t norm_kind; /* LCC_NORM_*: the block norms and the final norm (LCC_NORM_LAYER: sandwich blocks) */
     int32_t canon_taps; /* LCC_BLOCK_BRANCHNORM: taps of the convolution in front of every mixer (<= 8) */
     float final_norm_alpha; /* LCC_NORM_DYT */
     float logit_scale;      /* logits are multiplied by it (0 reads as 1) */

@@ -322,6 +322,7 @@ def seq_param_specs(cfg) -> List[Tuple[str, Tuple[int, ...], str]]:
     par = getattr(cfg, "block", "postnorm") == "parallel"     # one norm per layer
     dyt = getattr(cfg, "norm", "rms") == "dyt"                # a norm is a weight, a bias and a scalar
 
+    sandwich = getattr(cfg, "block", "postnorm") == "sandwich"   # a norm behind every sublayer too
     nshape = () if getattr(cfg, "norm_scalar", False) else (W,)      # a norm whose weight is one number
 
     def norm_specs(name):
@@ -334,14 +335,18 @@ def seq_param_specs(cfg) -> List[Tuple[str, Tuple[int, ...], str]]:
         specs += norm_specs(p + "norm1")
         if (L.ff or L.moe) and not par:
             specs.append((p + "norm2", nshape, norm))
+        if sandwich:
+            specs += [(p + n, nshape, norm) for n in (("norm1b", "norm2b") if (L.ff or L.moe) else ("norm1b",))]
         if getattr(cfg, "canon_taps", 0):
             specs.append((p + "canon1", (W, cfg.canon_taps), "canon"))
         if hc:
             n = cfg.streams
             for q in ("hc1.", "hc2.") if (L.ff or L.moe) else ("hc1.",):
                 specs += [(p + q + "in", (n,), "hc_in"), (p + q + "out", (n,), "hc_out"), (p + q + "mix", (n, n), "hc_mix")]
-        if L.type == "retention":
+        if L.type in ("retention", "lightning"):
             t, m = L.retention, p + "mix."
+            if t.whole_norm:
+                specs.append((m + "norm", (t.heads * t.vdim,), "norm"))
             specs += [(m + "q", (t.heads * t.dim, W), "w"), (m + "k", (t.heads * t.dim, W), "w"), (m + "v", (t.heads * t.vdim, W), "w"),
                       (m + "g", (t.heads * t.vdim, W), "w"), (m + "o", (W, t.heads * t.vdim), "w")]
         elif L.type == "channel_delta":
@@ -368,8 +373,14 @@ def seq_param_specs(cfg) -> List[Tuple[str, Tuple[int, ...], str]]:
             specs.append((m + "o", (W, a.heads * a.vdim), "w"))
         elif L.type == "attention":
             a, m = L.attn, p + "mix."
-            specs += [(m + "q", (a.heads * a.dim, W), "w"), (m + "k", (a.kv_heads * a.dim, W), "w")]
-            if not a.unit_norm:
+            specs += [(m + "q", (a.heads * a.maps * a.dim, W), "w"), (m + "k", (a.kv_heads * a.maps * a.dim, W), "w")]
+            if a.bias:
+                specs += [(m + "q.b", (a.heads * a.maps * a.dim,), "b"), (m + "k.b", (a.kv_heads * a.maps * a.dim,), "b")]
+                if not a.value_keys:
+                    specs.append((m + "v.b", (a.kv_heads * a.vdim,), "b"))
+            if a.maps > 1:
+                specs += [(m + n, (a.dim,), "lam") for n in ("lq1", "lk1", "lq2", "lk2")]
+            if a.qk_norm and not a.unit_norm:
                 specs += [(m + "q.norm", (a.dim,), "norm"), (m + "k.norm", (a.dim,), "norm")]
             if a.temp:
                 specs.append((m + "temp", (a.heads,), "skip"))
@@ -406,16 +417,17 @@ def seq_param_specs(cfg) -> List[Tuple[str, Tuple[int, ...], str]]:
                     specs.append((f"{m}e{j}.gate", (e.ff, W), "w"))
                 specs += [(f"{m}e{j}.up", (e.ff, W), "w"), (f"{m}e{j}.down", (W, e.ff), "w")]
             specs.append((m + "router", (e.outputs, W), "w"))
-            if e.router != "topk_softmax":
+            if e.router != "topk_softmax" and e.correction:
                 specs.append((m + "correction", (e.outputs,), "b"))
             if e.shared_ff:
-                specs += [(m + "shared.up", (e.shared_ff, W), "w"), (m + "shared.down", (W, e.shared_ff), "w"),
-                          (m + "shared.sg", (1, W), "w")]
+                specs += [(m + "shared.up", (e.shared_ff, W), "w"), (m + "shared.down", (W, e.shared_ff), "w")]
+                if e.shared_gate:
+                    specs.append((m + "shared.sg", (1, W), "w"))
         elif L.ff:
             if getattr(cfg, "dense", "glu") != "mlp":
                 specs.append((p + "mlp.gate", (L.ff, W), "w"))
             specs += [(p + "mlp.up", (L.ff, W), "w"), (p + "mlp.down", (W, L.ff), "w")]
-    specs += norm_specs("final.norm") + [("head", (cfg.vocab, W), "w")]
+    specs += norm_specs("final.norm") + ([] if getattr(cfg, "tied_head", False) else [("head", (cfg.vocab, W), "w")])
     return specs
 
 
@@ -449,6 +461,8 @@ def synthetic_seq_tensors(cfg, seed: int = 1234, device="cpu") -> Dict[str, torc
             t = u * 1.5
         elif kind == "canon":
             t = u * 0.8
+        elif kind == "lam":
+            t = u * (2.0 / shape[-1] ** 0.5)
         elif kind == "mix":
             t = 0.5 + 0.6 * u
         elif kind == "dt":

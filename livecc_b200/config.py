@@ -218,13 +218,19 @@ class RotaryConfig:
 
 @dataclass
 class RetentionConfig:
-    """Linear attention with one fixed decay per head and no normaliser: S <- decay_h S + k v^T, o = S^T q; rotary q and k,
-    k scaled by dim^-1/2; each head's output brought to unit rms, times silu(gate)."""
+    """Linear attention with one fixed decay per head and no normaliser: S <- decay_h S + k v^T, o = S^T q. The retention form:
+    rotary q and k, k scaled by dim^-1/2; each head's output brought to unit rms, times silu(gate). The lightning form (layer
+    type "lightning"): `silu` on q, k and v, no rotation, `key_scale` off, `whole_norm` (one RMS norm with a weight over all
+    heads together), gate "sigmoid"."""
     heads: int
     dim: int
     vdim: int
     decay: list
     rot: RotaryConfig
+    silu: bool = False
+    key_scale: bool = True
+    whole_norm: bool = False
+    gate: str = "silu"
 
 
 @dataclass
@@ -255,7 +261,9 @@ class MoeConfig:
     groups of neighbours, a group scores as its best choice score, and only members of the best `keep` groups can be chosen.
     `act`: "relu2" (down(relu(up x)^2)), "clamp_glu" (g = min(gate x, limit), u = clamp(up x, -limit, limit),
     down(g sigmoid(1.702 g) (u + 1))) or "silu_glu" (down(silu(gate x) * (up x))). `router` "topk_softmax": the `top` largest
-    logits are chosen and weighted by the softmax over the chosen logits only (no correction tensor)."""
+    logits are chosen and weighted by the softmax over the chosen logits only (no correction tensor). `act` "gelu": down(gelu(up x)),
+    the exact (erf) form. `group_top`: a group scores as the sum of that many of its best choice scores. `correction`: the
+    router has a correction tensor. `shared_gate`: the shared expert sits behind its gate (False: it is added as it is)."""
     experts: int
     top: int
     ff: int
@@ -267,6 +275,9 @@ class MoeConfig:
     keep: int = 0
     act: str = "relu2"
     limit: float = 0.0
+    group_top: int = 1
+    correction: bool = True
+    shared_gate: bool = True
 
     @property
     def outputs(self) -> int:
@@ -280,7 +291,12 @@ class MaskedAttnConfig:
     heads), rotary positions on the first rot.dims channels of a head (`rot_pairs`: channel 2i turns with 2i+1, else i with
     i + dims/2), a sliding window (row i sees j with 0 <= i - j < window; 0: none), `value_keys`: the values are the keys
     as projected, before norm and rotation (no value projection), `gate`: "none", "head" or "channel" (sigmoid of a
-    projection of the mixer's input, applied before the output projection), `sink`: a zero-logit term in the denominator."""
+    projection of the mixer's input, applied before the output projection), `sink`: a zero-logit term in the denominator.
+    `keep_first`: the first positions of the sequence stay visible behind the window. `softcap` > 0: scores become
+    softcap * tanh(score / softcap). `maps` = 2, differential attention: every query and key head is two maps of `dim` channels,
+    each with a softmax of its own over the same values; the second map's output times lambda is subtracted, lambda =
+    exp(lq1 . lk1) - exp(lq2 . lk2) + diff, the difference is brought to unit rms per head and multiplied by 1 - diff.
+    `qk_norm` False: q and k as projected. `bias`: q, k and v projections have biases."""
     heads: int
     kv_heads: int
     dim: int
@@ -294,6 +310,12 @@ class MaskedAttnConfig:
     sink: bool = False
     unit_norm: bool = False   # q and k heads are divided by their rms without a weight (no q.norm / k.norm tensors)
     temp: bool = False        # a learned factor per query head on the scores (tensor `temp`)
+    qk_norm: bool = True      # per-head RMS norm of q and k
+    bias: bool = False
+    maps: int = 1
+    diff: float = 0.0
+    softcap: float = 0.0
+    keep_first: int = 0
     v_mix: bool = False       # the cached values are (1 - vmix) v + vmix v_first, v_first = the first such layer's values of the token
 
     @property
@@ -323,12 +345,12 @@ class DeltaConfig:
 
 @dataclass
 class SeqLayerConfig:
-    type: str                      # "mamba2" | "parallel" | "retention" | "latent_attention" | "attention" | "channel_delta"
+    type: str                      # "mamba2" | "parallel" | "retention" | "lightning" | "latent_attention" | "attention" | "channel_delta"
     ssd: SsdMixerConfig = None
     left: ChunkAttnConfig = None
     right: GlaConfig = None
     ff: int = 0                    # 0 = the layer has no dense feed-forward
-    retention: RetentionConfig = None
+    retention: RetentionConfig = None   # types "retention" and "lightning"
     latent: LatentAttnConfig = None
     moe: MoeConfig = None          # routed feed-forward instead of the dense one
     attn: MaskedAttnConfig = None  # type "attention"
@@ -352,6 +374,14 @@ SEQ_FAMILIES = {
                     expert="silu_glu",
                     attention=dict(rot_pairs=False, value_keys=False, gate="none", sink=False, unit_norm=True, temp=True),
                     latent=dict(q_latent=True, gate=False, sink=False)),
+    # layer norms (weight, no bias) before and after every sublayer; differential attention with soft-capped scores inside a window
+    # that keeps the first tokens, no positions; lightning attention; two-matrix squared-relu feed-forward; sigmoid router without
+    # correction whose groups score as the sum of their two best, exact-gelu experts, an ungated shared expert; the head is the
+    # embedding table
+    "Kapitar": dict(block="sandwich", norm_offset=0.0, positions=None, norm="layer", dense="mlp", dense_act="relu2", router="sigmoid",
+                    expert="gelu", group_top=2, correction=False, shared_gate=False, tied_head=True,
+                    attention=dict(rot_pairs=False, value_keys=False, gate="none", sink=False, qk_norm=False, bias=True, maps=2),
+                    lightning=dict(silu=True, key_scale=False, whole_norm=True, gate="sigmoid")),
 }
 
 
@@ -367,11 +397,14 @@ class SeqModelConfig:
     logit_softcap: float = 0.0
     eos_token_id: int = -1         # none unless config.json names one
     block: str = "postnorm"        # "postnorm" | "prenorm_hc" (pre-norm sublayers on `streams` residual streams) | "parallel" |
-                                   # "branchnorm" (x <- x + norm(sublayer(x)); the mixer reads x + conv(x) when canon_taps > 0)
+                                   # "branchnorm" (x <- x + norm(sublayer(x)); the mixer reads x + conv(x) when canon_taps > 0) |
+                                   # "sandwich" (x <- x + normb(sublayer(norm(x))))
     canon_taps: int = 0            # taps of the causal convolution over time in front of every mixer (tensor l<i>.canon1 [width, taps])
     norm_scalar: bool = False      # a norm's weight is ONE number (tensors of one element)
-    norm: str = "rms"              # "rms" | "dyt" (tanh(alpha x) w + b; tensors <name>, <name>.b, <name>.alpha)
-    dense: str = "glu"             # dense feed-forward: "glu" (gelu_tanh(gate) * up) | "mlp" (gelu_tanh(up))
+    norm: str = "rms"              # "rms" | "dyt" (tanh(alpha x) w + b; tensors <name>, <name>.b, <name>.alpha) | "layer" (mean taken off, no bias)
+    dense: str = "glu"             # dense feed-forward: "glu" (gelu_tanh(gate) * up) | "mlp" (dense_act(up))
+    dense_act: str = "gelu_tanh"   # activation of a two-matrix feed-forward: "gelu_tanh" | "relu2"
+    tied_head: bool = False        # the output head is the embedding table
     logit_scale: float = 1.0
     streams: int = 1
     norm_offset: float = 0.0       # added to every stored layer-norm weight (1.0: weights stored around zero)
@@ -398,7 +431,9 @@ class SeqModelConfig:
                                     scale=float(r.get("scale", 1.0)), shared_ff=int(sh["ff"]) if sh else 0,
                                     router=fam.get("router", "sigmoid"), identity=int(r.get("identity", 0)),
                                     groups=int(gr["count"]) if gr else 0, keep=int(gr["keep"]) if gr else 0,
-                                    act=fam.get("expert", "relu2"), limit=float(mlp["expert"].get("limit", 0.0)))
+                                    act=fam.get("expert", "relu2"), limit=float(mlp["expert"].get("limit", 0.0)),
+                                    group_top=int(fam.get("group_top", 1)), correction=bool(fam.get("correction", True)),
+                                    shared_gate=bool(fam.get("shared_gate", True)))
                 else:
                     raise NotImplementedError(f"layer {i}: feed-forward kind {kind!r} is not supported")
             share = L.get("weights_of")
@@ -417,15 +452,23 @@ class SeqModelConfig:
                 if "attention" not in fam:
                     raise NotImplementedError(f"layer {i}: {arch} has no mixer of type 'attention'")
                 rot = RotaryConfig.from_json(mx["rot"]) if mx.get("rot") else RotaryConfig(0, 10000.0)
+                mask = mx.get("mask") or {}
                 layers.append(SeqLayerConfig("attention", ff=ff, moe=moe, weights_of=-1 if share is None else share, attn=MaskedAttnConfig(
                     heads=int(mx["heads"]), kv_heads=int(mx.get("kv_heads", mx["heads"])), dim=int(mx["dim"]),
-                    vdim=int(mx.get("vdim", mx["dim"])), window=int((mx.get("mask") or {}).get("size", 0)),
+                    vdim=int(mx.get("vdim", mx["dim"])), window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0),
+                    softcap=float(mx.get("softcap") or 0.0), diff=float(mx.get("diff", 0.0)),
                     scale=float(mx.get("scale", float(mx["dim"]) ** -0.5)), rot=rot, v_mix=bool(mx.get("v_mix", False)), **fam["attention"])))
             elif L["type"] == "channel_delta":
                 layers.append(SeqLayerConfig("channel_delta", ff=ff, moe=moe, delta=DeltaConfig(
                     heads=int(mx["heads"]), kv_heads=int(mx.get("kv_heads", mx["heads"])), dim=int(mx["dim"]),
                     vdim=int(mx.get("vdim", mx["dim"])), conv=int(mx.get("conv", 4)), rank_a=int(mx.get("decay_rank", 0)),
                     rank_g=int(mx.get("gate_rank", 0)))))
+            elif L["type"] == "lightning":
+                if "lightning" not in fam:
+                    raise NotImplementedError(f"layer {i}: {arch} has no mixer of type 'lightning'")
+                layers.append(SeqLayerConfig("lightning", ff=ff, moe=moe, retention=RetentionConfig(
+                    heads=int(mx["heads"]), dim=int(mx["dim"]), vdim=int(mx.get("vdim", mx["dim"])),
+                    decay=[float(x) for x in mx["decay"]], rot=RotaryConfig(0, 10000.0), **fam["lightning"])))
             elif L["type"] == "retention":
                 rot = RotaryConfig.from_json(mx["rot"]) if mx.get("rot") else RotaryConfig(0, 10000.0)
                 layers.append(SeqLayerConfig("retention", ff=ff, moe=moe, retention=RetentionConfig(
@@ -460,7 +503,7 @@ class SeqModelConfig:
             eos_token_id=int(d.get("eos_token_id", -1)), block=fam["block"], streams=int(d.get("streams", 1)),
             norm_offset=fam["norm_offset"], positions=fam["positions"], norm=fam.get("norm", "rms"), dense=fam.get("dense", "glu"),
             logit_scale=float(d.get("logit_scale", 1.0)), canon_taps=int((d.get("canon") or {}).get("taps", 0)),
-            norm_scalar=bool(fam.get("norm_scalar", False)))
+            norm_scalar=bool(fam.get("norm_scalar", False)), dense_act=fam.get("dense_act", "gelu_tanh"), tied_head=bool(fam.get("tied_head", False)))
 
     def to_json(self) -> dict:
         """The inverse of from_json (used to write synthetic checkpoints)."""
@@ -469,6 +512,9 @@ class SeqModelConfig:
             if L.type == "mamba2":
                 s = L.ssd
                 mx = dict(heads=s.heads, vdim=s.vdim, state=s.state, groups=s.groups, conv=s.conv, norm_groups=s.norm_groups)
+            elif L.type == "lightning":
+                t = L.retention
+                mx = dict(heads=t.heads, dim=t.dim, vdim=t.vdim, decay=list(t.decay))
             elif L.type == "retention":
                 t = L.retention
                 mx = dict(heads=t.heads, dim=t.dim, vdim=t.vdim, decay=list(t.decay), rot=t.rot.to_json())
@@ -484,8 +530,16 @@ class SeqModelConfig:
             elif L.type == "attention":
                 a = L.attn
                 mx = dict(heads=a.heads, kv_heads=a.kv_heads, dim=a.dim, vdim=a.vdim, scale=a.scale, rot=a.rot.to_json())
+                if not a.rot.dims and a.maps > 1:
+                    del mx["rot"]
                 if a.window:
                     mx["mask"] = dict(size=a.window)
+                    if a.keep_first:
+                        mx["mask"]["keep_first"] = a.keep_first
+                if a.softcap:
+                    mx["softcap"] = a.softcap
+                if a.maps > 1:
+                    mx["diff"] = a.diff
                 if a.v_mix:
                     mx["v_mix"] = True
             elif L.type == "channel_delta":
@@ -516,6 +570,8 @@ class SeqModelConfig:
             out.append(dict(type=L.type, mixer=mx, mlp=mlp))
             if L.weights_of >= 0:
                 out[-1]["weights_of"] = L.weights_of
+        if self.block == "sandwich":
+            return dict(architecture=self.architecture, vocab=self.vocab, width=self.width, layers=out, norm=dict(eps=self.eps))
         if self.block == "branchnorm":
             out_d = dict(architecture=self.architecture, vocab=self.vocab, width=self.width, layers=out, norm=dict(eps=self.eps))
             if self.canon_taps:
@@ -556,8 +612,10 @@ class SeqModelConfig:
                 continue
             if L.type == "attention":
                 a = L.attn
-                if self.block not in ("parallel", "branchnorm"):
+                if self.block not in ("parallel", "branchnorm", "sandwich"):
                     raise ValueError(f"layer {i}: the attention mixer is served in parallel blocks and in blocks normed on the sublayer's output")
+                if a.maps not in (1, 2) or a.keep_first < 0 or a.softcap < 0 or a.vdim < 1:
+                    raise ValueError(f"layer {i}: unsupported attention options {a}")
                 if a.v_mix:
                     first = next(x.attn for x in self.layers if x.type == "attention" and x.attn.v_mix)
                     if a.value_keys or (first.kv_heads, first.vdim) != (a.kv_heads, a.vdim):
@@ -570,7 +628,7 @@ class SeqModelConfig:
                 s = L.ssd
                 if s.heads % s.groups or s.inner % s.norm_groups or not 1 <= s.conv <= 8 or s.state > 512:
                     raise ValueError(f"layer {i}: unsupported state-space sizes {s}")
-            elif L.type == "retention":
+            elif L.type in ("retention", "lightning"):
                 t = L.retention
                 if len(t.decay) != t.heads or t.dim > 512 or t.rot.dims % 2 or t.rot.dims > t.dim or \
                         any(not 0.0 < x <= 1.0 for x in t.decay):

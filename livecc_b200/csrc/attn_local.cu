@@ -2,7 +2,8 @@
 //   * q/k RMS norm over the whole projection (all heads at once) and the append of k, v to the pages,
 //   * attention of new rows over the keys of their own chunk (chunks counted from position 0 of the sequence) with a
 //     softmax sink: p_j = exp(s_j) / (exp(sink_h) + sum_j exp(s_j)) (sink_h = 0 unless given), and a per-head sigmoid output gate.
-// Options (AttnOpts): a sliding window instead of / inside the chunks, no sink (ordinary softmax), one gate per output channel.
+// Options (AttnOpts): a sliding window instead of / inside the chunks that may keep the first positions, no sink (ordinary softmax),
+// one gate per output channel, soft-capped scores, two maps per head whose difference is the output (differential attention).
 // Scores, weights and the accumulation are fp32; K and V pages hold the model's storage type.
 #include <math.h>
 #include <stdlib.h>
@@ -32,6 +33,21 @@ __device__ __forceinline__ int first_key(int p, int chunk, int window) {
     int lo = chunk > 0 ? (p / chunk) * chunk : 0;
     if (window > 0) lo = max(lo, p - window + 1);
     return lo;
+}
+// cap * tanh(s / cap), a score's soft cap
+__device__ __forceinline__ float soft_cap(float s, float cap, float inv_cap) { return cap * tanhf(s * inv_cap); }
+// The same through one exponential and one reciprocal, for the bf16 tensor-core kernel: tanh(y) = 1 - 2 / (1 + e^(2y)). The absolute
+// error stays near cap * 2^-22, which is what a softmax sees; e^(2y) past the fp32 range gives +-1.
+__device__ __forceinline__ float soft_cap_fast(float s, float cap, float inv_cap) {
+    const float e = __expf(2.f * fminf(s * inv_cap, 40.f));
+    return cap - __fdividef(2.f * cap, 1.f + e);
+}
+// With a window that keeps the first `keep` positions, a row whose window starts at `lo` sees [0, keep) and [lo, p]. The key tiles of
+// a group of rows whose first window starts at `kbeg` are walked from `k_start` on; a step from a tile of the kept positions skips
+// what lies between them and kbeg.
+__device__ __forceinline__ int next_tile(int kc, int step, int keep, int kbeg) {
+    const int n = kc + step;
+    return (n >= keep && n < kbeg) ? kbeg : n;
 }
 // A softmax without a sink starts its running (max, sum) at (kNoSinkMax, 0): finite, so that a tile in which a row sees no
 // key leaves both unchanged (exp(-inf - kNoSinkMax) = 0) and the first visible key rescales the empty sum by exp(-huge) = 0.
@@ -188,7 +204,8 @@ __global__ void __launch_bounds__(128) attn_chunk_sink_kernel(const float* __res
     const int g = h / (Hq / G);
     const int p = seq_past(pos, S) + t;
     const int start = first_key(p, chunk, opt.window);
-    const int nkeys = p - start + 1;
+    const int nkeep = min(opt.keep_first, start), nkeys = p - start + 1 + nkeep;   // key jk: the kept positions, then the window's
+    const int ld_k = D * opt.maps, koff = (h % opt.maps) * D;
     float* sq = sm;           // [D]
     float* sc = sm + D;       // [nkeys]
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
@@ -197,11 +214,12 @@ __global__ void __launch_bounds__(128) attn_chunk_sink_kernel(const float* __res
     // scores: one warp per key, lanes over the head dimension
     float mx = sk;  // the sink's score
     for (int jk = warp; jk < nkeys; jk += nwarps) {
-        const int pj = start + jk;
-        const T* kr = k_pages + (((size_t)page_table[pj / page_size] * G + g) * page_size + pj % page_size) * D;
+        const int pj = jk < nkeep ? jk : start + jk - nkeep;
+        const T* kr = k_pages + (((size_t)page_table[pj / page_size] * G + g) * page_size + pj % page_size) * ld_k + koff;
         float acc = 0.f;
         for (int d = lane; d < D; d += 32) acc = fmaf(sq[d], ldf(kr + d), acc);
         acc = warp_sum(acc) * scale;
+        if (opt.softcap > 0.f) acc = soft_cap(acc, opt.softcap, 1.f / opt.softcap);
         if (lane == 0) sc[jk] = acc;
         mx = fmaxf(mx, acc);
     }
@@ -222,10 +240,11 @@ __global__ void __launch_bounds__(128) attn_chunk_sink_kernel(const float* __res
     for (int c = threadIdx.x; c < DV; c += blockDim.x) {
         float acc = 0.f;
         for (int jk = 0; jk < nkeys; ++jk) {
-            const int pj = start + jk;
+            const int pj = jk < nkeep ? jk : start + jk - nkeep;
             const T* vr = v_pages + (((size_t)page_table[pj / page_size] * G + g) * page_size + pj % page_size) * ld_v;
             acc = fmaf(sc[jk], ldf(vr + c), acc);
         }
+        if (opt.raw) { opt.raw[((size_t)t * Hq + h) * DV + c] = acc * inv; continue; }
         const float gv = gate ? gate_of(gate, ld_gate, t, h, c, DV, opt.gate_channel) : 1.f;
         stf(out + (size_t)t * ld_out + (size_t)h * DV + c, acc * inv * gv);
     }
@@ -236,7 +255,9 @@ __global__ void __launch_bounds__(128) attn_chunk_sink_kernel(const float* __res
 // split + n_splits, ... of kSplitKeys keys each (so any length works with any grid; the grid only sets the parallelism), keeps
 // the running (max, sum, output) over its tiles, and leaves them in the workspace; the CTA that arrives last at the
 // (row, head) counter merges the splits with the sink's term, applies the gate and writes the row. The counter goes back to
-// zero for the next launch.
+// zero for the next launch. With two maps per head (opt.maps = 2) the grid has one CTA per (row, head, map, split), the
+// counter is the head's, and the last CTA merges both maps and writes their normed difference.
+// Keys are numbered as the row sees them: the kept first positions, then the window's.
 constexpr int kSplitKeys = 128, kSplitMaxOut = 4;   // output channels per thread: DV <= 128 * kSplitMaxOut
 // The arrival counters take a fixed area at the head of the workspace, whatever the row and head counts of a call: partials
 // of one call must never lie where another call (a layer with other sizes) keeps its counters.
@@ -274,10 +295,11 @@ __global__ void __launch_bounds__(128) attn_split_kernel(const float* __restrict
     float* sq = sm;            // [D]
     float* sc = sm + D;        // [kSplitKeys]
     const int t = blockIdx.y, h = blockIdx.x, z = blockIdx.z, nz = gridDim.z;
-    const int g = h / (Hq / G);
-    const int nkeys = seq_past(pos, S) + t + 1;
-    // with a window the walk starts at the tile that holds the row's first key; keys of that tile before it are masked
-    const int kfirst = first_key(nkeys - 1, 0, opt.window), tile0 = kfirst / kSplitKeys;
+    const int g = h / (Hq / G);                  // (Hq counts the maps too)
+    const int npos = seq_past(pos, S) + t + 1;
+    const int kfirst = first_key(npos - 1, 0, opt.window), nkeep = min(opt.keep_first, kfirst), nkeys = npos - kfirst + nkeep;
+    const int ld_k = D * opt.maps, koff = (h % opt.maps) * D;
+    const float inv_cap = opt.softcap > 0.f ? 1.f / opt.softcap : 0.f;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     for (int i = threadIdx.x; i < D; i += blockDim.x) sq[i] = q[((size_t)t * Hq + h) * D + i] * scale;
     float m = -INFINITY, l = 0.f;
@@ -285,12 +307,12 @@ __global__ void __launch_bounds__(128) attn_split_kernel(const float* __restrict
     constexpr int VN = VEC ? RowVec<T>::N : 1, NP = VEC ? 128 * kSplitMaxOut / (32 * RowVec<T>::N) : 1;
     float ov[NP][VN] = {};                           // vector form: a warp's sum over ITS keys of 16-byte pieces lane, lane + 32, ...
     float* osum = sc + kSplitKeys;                   // [4][DV], vector form only
-    for (int k0 = (tile0 + z) * kSplitKeys; k0 < nkeys; k0 += nz * kSplitKeys) {
+    for (int k0 = z * kSplitKeys; k0 < nkeys; k0 += nz * kSplitKeys) {
         const int nk = min(kSplitKeys, nkeys - k0);
         __syncthreads();       // sq is staged; the previous tile's weights are consumed
         // every key's row in the page pool first (one page-table read per thread, all in flight together)
         for (int j = threadIdx.x; j < nk; j += blockDim.x) {
-            const int pj = k0 + j;
+            const int pj = k0 + j < nkeep ? k0 + j : kfirst + k0 + j - nkeep;
             row_of[j] = (int)(((size_t)page_table[pj / page_size] * G + g) * page_size + pj % page_size);
         }
         __syncthreads();
@@ -300,7 +322,7 @@ __global__ void __launch_bounds__(128) attn_split_kernel(const float* __restrict
         for (int j0 = warp * KG; j0 < nk; j0 += 4 * KG) {
             const T* kr[KG];
 #pragma unroll
-            for (int j = 0; j < KG; ++j) kr[j] = k_pages + (size_t)row_of[min(j0 + j, nk - 1)] * D;
+            for (int j = 0; j < KG; ++j) kr[j] = k_pages + (size_t)row_of[min(j0 + j, nk - 1)] * ld_k + koff;
             float acc[KG];
 #pragma unroll
             for (int j = 0; j < KG; ++j) acc[j] = 0.f;
@@ -327,7 +349,7 @@ __global__ void __launch_bounds__(128) attn_split_kernel(const float* __restrict
 #pragma unroll
             for (int j = 0; j < KG; ++j) {
                 float v = warp_sum(acc[j]);
-                if (k0 + j0 + j < kfirst) v = -INFINITY;       // before the window (first tile only)
+                if (opt.softcap > 0.f) v = soft_cap(v, opt.softcap, inv_cap);
                 if (j0 + j < nk) {
                     if (lane == 0) sc[j0 + j] = v;
                     mx = fmaxf(mx, v);
@@ -416,10 +438,42 @@ __global__ void __launch_bounds__(128) attn_split_kernel(const float* __restrict
     }
     __threadfence();
     __syncthreads();
-    if (threadIdx.x == 0) last_flag = atomicAdd(counters + t * Hq + h, 1) == nz - 1;
+    int* counter = counters + t * (Hq / opt.maps) + h / opt.maps;
+    if (threadIdx.x == 0) last_flag = atomicAdd(counter, 1) == nz * opt.maps - 1;
     __syncthreads();
     if (!last_flag) return;
     __threadfence();
+    if (opt.maps == 2) {
+        // both maps of the head are complete: o = a1 - lambda a2, brought to unit rms over the head's channels, times the scale
+        const int hd = h >> 1;
+        float ov2[kSplitMaxOut] = {}, ss = 0.f;
+        for (int mp = 0; mp < 2; ++mp) {
+            const float* pm = part + ((size_t)t * Hq + 2 * hd + mp) * nz * (DV + 2);
+            float mt = -INFINITY, lt = 0.f;
+            for (int i = 0; i < nz; ++i) mt = fmaxf(mt, __ldcg(pm + (size_t)i * (DV + 2)));   // split 0 holds a key: finite
+            for (int i = 0; i < nz; ++i) lt = fmaf(__ldcg(pm + (size_t)i * (DV + 2) + 1), expf(__ldcg(pm + (size_t)i * (DV + 2)) - mt), lt);
+            const float f = (mp ? -opt.lambda : 1.f) / lt;
+            for (int i = 0; i < nz; ++i) {
+                const float w = expf(__ldcg(pm + (size_t)i * (DV + 2)) - mt) * f;
+#pragma unroll
+                for (int u = 0; u < kSplitMaxOut; ++u) {
+                    const int c = threadIdx.x + u * 128;
+                    if (c < DV) ov2[u] = fmaf(__ldcg(pm + (size_t)i * (DV + 2) + 2 + c), w, ov2[u]);
+                }
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < kSplitMaxOut; ++u) ss = fmaf(ov2[u], ov2[u], ss);
+        ss = block_sum(ss, red);
+        const float rn = opt.diff_scale / sqrtf(ss / (float)DV + opt.eps);
+#pragma unroll
+        for (int u = 0; u < kSplitMaxOut; ++u) {
+            const int c = threadIdx.x + u * 128;
+            if (c < DV) stf(out + (size_t)t * ld_out + (size_t)hd * DV + c, ov2[u] * rn);
+        }
+        if (threadIdx.x == 0) *counter = 0;
+        return;
+    }
     const float* all = part + ((size_t)t * Hq + h) * nz * (DV + 2);
     const float sk = opt.no_sink ? -INFINITY : (sink ? sink[h] : 0.f);   // split 0 holds the row's first key: mt is finite
     float mt = sk;
@@ -434,7 +488,7 @@ __global__ void __launch_bounds__(128) attn_split_kernel(const float* __restrict
         const float gv = gate ? gate_of(gate, ld_gate, t, h, c, DV, opt.gate_channel) : 1.f;
         stf(out + (size_t)t * ld_out + (size_t)h * DV + c, acc * f * gv);
     }
-    if (threadIdx.x == 0) counters[t * Hq + h] = 0;
+    if (threadIdx.x == 0) *counter = 0;
 }
 
 // Prompt portions: one CTA per (64 query rows, query head, 128 output channels). Keys are walked in tiles of 64 from the
@@ -484,6 +538,9 @@ __global__ void __launch_bounds__(256) attn_chunk_sink_tiled_kernel(const float*
     const int rows = min(AQ, S - t0);
     const int pf = past + t0, pl = pf + rows - 1;
     const int kbeg = first_key(pf, chunk, opt.window);       // the first row's first key: no later row starts earlier
+    const int keep = min(opt.keep_first, kbeg), k_start = keep > 0 ? 0 : kbeg;
+    const int ld_k = D * opt.maps, koff = (h % opt.maps) * D;
+    const float inv_cap = opt.softcap > 0.f ? 1.f / opt.softcap : 0.f;
     const int tm = (threadIdx.x / 16) * 4, tn = (threadIdx.x % 16) * 4;
     const int lr = threadIdx.x / 16, lc = threadIdx.x % 16;              // staging: 16 threads walk a row
     int p_row[4], lo_row[4];
@@ -499,13 +556,15 @@ __global__ void __launch_bounds__(256) attn_chunk_sink_tiled_kernel(const float*
     const float* qh = q + ((size_t)t0 * Hq + h) * D;
     const bool q_once = D <= ADC;
     bool q_staged = false;
-    for (int k0 = kbeg; k0 <= pl; k0 += AK) {
+    for (int k0 = k_start; k0 <= pl; k0 = next_tile(k0, AK, keep, kbeg)) {
         const int nk = min(AK, pl - k0 + 1);
+        bool row_ok[4];
         size_t row_off[4];                               // this thread's 4 key rows of the tile, as (page, group, slot) bases
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int pj = k0 + lr + 16 * j;
-            row_off[j] = pj <= pl ? ((size_t)page_table[pj / page_size] * G + g) * page_size + pj % page_size : 0;
+            row_ok[j] = pj <= pl && (pj >= kbeg || pj < keep);   // (between the kept positions and the window lies no visible key)
+            row_off[j] = row_ok[j] ? ((size_t)page_table[pj / page_size] * G + g) * page_size + pj % page_size : 0;
         }
         float sc[4][4] = {};
         for (int d0 = 0; d0 < D; d0 += ADC) {
@@ -521,8 +580,8 @@ __global__ void __launch_bounds__(256) attn_chunk_sink_tiled_kernel(const float*
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int r = lr + 16 * j;
-                const T* kr = k_pages + row_off[j] * D + d0;
-                if (r < nk) {
+                const T* kr = k_pages + row_off[j] * ld_k + koff + d0;
+                if (row_ok[j]) {
 #pragma unroll 8
                     for (int d = lc; d < dn; d += 16) sk_[d * APQ + r] = kr[d];
                 } else {
@@ -536,7 +595,7 @@ __global__ void __launch_bounds__(256) attn_chunk_sink_tiled_kernel(const float*
                     const T* vr = v_pages + row_off[j] * ld_v + c0;
                     if (r < nk) {
 #pragma unroll 8
-                        for (int c = lc; c < AVW; c += 16) sv_[r * APV + c] = c0 + c < DV ? vr[c] : T(0.f);
+                        for (int c = lc; c < AVW; c += 16) sv_[r * APV + c] = (row_ok[j] && c0 + c < DV) ? vr[c] : T(0.f);
                     }
                 }
             }
@@ -560,8 +619,9 @@ __global__ void __launch_bounds__(256) attn_chunk_sink_tiled_kernel(const float*
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int pj = k0 + tn + j;
-                const bool ok = pj <= p_row[i] && pj >= lo_row[i] && tm + i < rows;
-                sc[i][j] = ok ? sc[i][j] * scale : -INFINITY;
+                const bool ok = pj <= p_row[i] && (pj >= lo_row[i] || pj < opt.keep_first) && tm + i < rows;
+                const float v = sc[i][j] * scale;
+                sc[i][j] = ok ? (opt.softcap > 0.f ? soft_cap(v, opt.softcap, inv_cap) : v) : -INFINITY;
                 mx = fmaxf(mx, sc[i][j]);
             }
 #pragma unroll
@@ -608,6 +668,7 @@ __global__ void __launch_bounds__(256) attn_chunk_sink_tiled_kernel(const float*
         for (int c = 0; c < 8; ++c) {
             const int col = c0 + (c < 4 ? tn + c : 64 + tn + c - 4);
             if (col < DV) {
+                if (opt.raw) { opt.raw[((size_t)t * Hq + h) * DV + col] = o[i][c] * f; continue; }
                 const float gv = gate ? gate_of(gate, ld_gate, t, h, col, DV, opt.gate_channel) : 1.f;
                 stf(out + (size_t)t * ld_out + (size_t)h * DV + col, o[i][c] * f * gv);
             }
@@ -641,8 +702,8 @@ constexpr int MQ = 64, MK = 64;
 
 // rows that are not 16-byte aligned: element-wise staging
 template <typename RowPtr>
-__device__ __forceinline__ void stage_bf16_rows(bf16* dst, int ld_dst, int ncp, int ncv, RowPtr rowptr) {
-    for (int u = threadIdx.x; u < MK * ncp; u += blockDim.x) {
+__device__ __forceinline__ void stage_bf16_rows(bf16* dst, int n_rows, int ld_dst, int ncp, int ncv, RowPtr rowptr) {
+    for (int u = threadIdx.x; u < n_rows * ncp; u += blockDim.x) {
         const int r = u / ncp, c = u % ncp;
         const bf16* p = rowptr(r);
         dst[(size_t)r * ld_dst + c] = (p && c < ncv) ? p[c] : __float2bfloat16_rn(0.f);
@@ -651,8 +712,11 @@ __device__ __forceinline__ void stage_bf16_rows(bf16* dst, int ld_dst, int ncp, 
 
 // NBUF (VEC8 only): 2 = the next tile's copies fly while this one is computed; 1 = one buffer, which halves the shared memory so
 // that two CTAs share an SM and hide each other's copies and tensor-pipe latency instead.
-template <bool VEC8, int KH, int NV, int NBUF = 2>
-__global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1) ? 2 : 0) attn_chunk_sink_mma_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pages,
+// MAPS = 2 (differential attention; KH = 2): the two groups of warps take the two maps of one head over the SAME key tiles, so a tile's
+// V rows are staged once for both; at the end the second group hands its normalised output to the first, which writes the normed
+// difference. D is a map's width; key rows hold both maps.
+template <bool VEC8, int KH, int NV, int NBUF = 2, int MAPS = 1>
+__global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 : 0) attn_chunk_sink_mma_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pages,
                                                                   const bf16* __restrict__ v_pages, const int* __restrict__ page_table,
                                                                   int page_size, const bf16* __restrict__ gate, int ld_gate,
                                                                   bf16* __restrict__ out, int ld_out, int S, int Hq, int G, int D, int DV,
@@ -663,24 +727,30 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1) ? 2 : 0) attn_ch
     // NV output tiles of 128 channels per CTA (NV = 2: values of up to 256 channels against one pass over the scores)
     constexpr int MVW = 128 * NV, MLV = MVW + 8;
     const int Dp = (D + 15) / 16 * 16, LQ = Dp + 8;
-    bf16* sQ = reinterpret_cast<bf16*>(smem_attn);     // [MQ][LQ]
-    constexpr int KT = KH * MK;                         // keys per step of the CTA: one 64-key tile per group of 4 warps
-    bf16* sK0 = sQ + (size_t)MQ * LQ;                   // [2][KT][LQ]   (the second buffer only with VEC8)
-    bf16* sV0 = sK0 + (size_t)(VEC8 ? NBUF : 1) * KT * LQ; // [2][KT][MLV]
+    static_assert(MAPS == 1 || KH == 2, "one group of warps per map");
+    bf16* sQ = reinterpret_cast<bf16*>(smem_attn);     // [MAPS][MQ][LQ]
+    constexpr int KT = MAPS == 2 ? MK : KH * MK;        // keys per step of the CTA: one 64-key tile per group of 4 warps (two maps: one for both)
+    constexpr int KR = MAPS * KT;                       // K rows of a buffer (the second map's tile behind the first's)
+    bf16* sK0 = sQ + (size_t)MAPS * MQ * LQ;            // [2][MAPS][KT][LQ]   (the second buffer only with VEC8)
+    bf16* sV0 = sK0 + (size_t)(VEC8 ? NBUF : 1) * KR * LQ; // [2][KT][MLV]
     const int t0 = (gridDim.y - 1 - blockIdx.y) * MQ, h = blockIdx.x, c0 = blockIdx.z * MVW;
     const int g = h / (Hq / G);
     const int past = seq_past(pos, S);
     const int rows = min(MQ, S - t0);
     const int pf = past + t0, pl = pf + rows - 1;
     const int kbeg = first_key(pf, chunk, opt.window);       // the first row's first key: no later row starts earlier
+    const int keep = min(opt.keep_first, kbeg), k_start = keep > 0 ? 0 : kbeg;
+    // a CTA of one map works on head h = head * opt.maps + map (its K columns start at map * D), a CTA of both maps on head h
+    const int ld_k = D * opt.maps, koff = MAPS == 1 ? (h % opt.maps) * D : 0;
+    const float inv_cap = opt.softcap > 0.f ? 1.f / opt.softcap : 0.f;
     const int dvv = min(MVW, DV - c0), DVp = (dvv + 15) / 16 * 16;
     const int warp = (threadIdx.x >> 5) & 3, kh = threadIdx.x >> 7, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
     // queries: fp32 -> bf16, zero padding
-    for (int u = threadIdx.x; u < MQ * (Dp / 2); u += blockDim.x) {
-        const int r = u / (Dp / 2), d = (u % (Dp / 2)) * 2;
-        const float* qr = q + ((size_t)(t0 + r) * Hq + h) * D;
+    for (int u = threadIdx.x; u < MAPS * MQ * (Dp / 2); u += blockDim.x) {
+        const int rm = u / (Dp / 2), d = (u % (Dp / 2)) * 2, r = MAPS == 2 ? rm % MQ : rm;
+        const float* qr = q + ((size_t)(t0 + r) * Hq * MAPS + (MAPS == 2 ? 2 * h + rm / MQ : h)) * D;
         const float v0 = (r < rows && d < D) ? qr[d] : 0.f, v1 = (r < rows && d + 1 < D) ? qr[d + 1] : 0.f;
-        *reinterpret_cast<uint32_t*>(sQ + (size_t)r * LQ + d) = pack_bf16x2(v0, v1);
+        *reinterpret_cast<uint32_t*>(sQ + (size_t)rm * LQ + d) = pack_bf16x2(v0, v1);
     }
     const int r_lo = warp * 16 + gq;                    // this thread's two rows of the tile: r_lo and r_lo + 8
     int p_row[2], lo_row[2];
@@ -692,27 +762,27 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1) ? 2 : 0) attn_ch
     const float sk = opt.no_sink ? kNoSinkMax : (sink ? sink[blockIdx.x] : 0.f);
     float m[2] = {sk, sk};
     // per-thread partial sums; the sink's 1 is counted once per row (by one thread of the first group of warps)
-    const float l0 = (tq == 0 && kh == 0 && !opt.no_sink) ? 1.f : 0.f;
+    const float l0 = (tq == 0 && (kh == 0 || MAPS == 2) && !opt.no_sink) ? 1.f : 0.f;
     float l[2] = {l0, l0};
     float o[16 * NV][4] = {};
     // VEC8: a tile's K and V rows arrive by 16-byte asynchronous copies (zero-filled past the last key and in the padding
     // columns), all in flight together, into the buffer the previous tile does not use, while that tile is computed
     auto issue = [&](int k0, int buf) {
-        bf16* dK = sK0 + (size_t)buf * KT * LQ;
+        bf16* dK = sK0 + (size_t)buf * KR * LQ;
         bf16* dV = sV0 + (size_t)buf * KT * MLV;
         // a warp walks rows, its lanes walk a row's 16-byte pieces; page and slot advance without divisions
-        const int kpr = Dp / 8, vpr = DVp / 8, nw = blockDim.x >> 5, wid = threadIdx.x >> 5;
+        const int kpr = Dp / 8, kpm = MAPS * kpr, vpr = DVp / 8, nw = blockDim.x >> 5, wid = threadIdx.x >> 5;
         int pj = k0 + wid, pg = pj / page_size, slot = pj - pg * page_size;
         for (int r = wid; r < KT; r += nw) {
-            const bool row_ok = pj <= pl;
+            const bool row_ok = pj <= pl && (pj >= kbeg || pj < keep);
             const size_t ro = row_ok ? ((size_t)page_table[pg] * G + g) * page_size + slot : 0;
-            for (int cu = lane; cu < kpr + vpr; cu += 32) {
-                if (cu < kpr) {
-                    const int c = cu * 8;
+            for (int cu = lane; cu < kpm + vpr; cu += 32) {
+                if (cu < kpm) {
+                    const int mp = MAPS == 2 && cu >= kpr ? 1 : 0, c = (cu - mp * kpr) * 8;
                     const bool ok = row_ok && c < D;
-                    cp_async16(dK + (size_t)r * LQ + c, ok ? k_pages + ro * D + c : k_pages, ok);
+                    cp_async16(dK + ((size_t)mp * KT + r) * LQ + c, ok ? k_pages + ro * ld_k + koff + mp * D + c : k_pages, ok);
                 } else {
-                    const int c = (cu - kpr) * 8;
+                    const int c = (cu - kpm) * 8;
                     const bool ok = row_ok && c < dvv;
                     cp_async16(dV + (size_t)r * MLV + c, ok ? v_pages + ro * ld_v + c0 + c : v_pages, ok);
                 }
@@ -722,13 +792,13 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1) ? 2 : 0) attn_ch
         }
         cp_async_commit();
     };
-    if (VEC8 && NBUF == 2) issue(kbeg, 0);
+    if (VEC8 && NBUF == 2) issue(k_start, 0);
     int it = 0;
-    for (int kc = kbeg; kc <= pl; kc += KT, ++it) {
+    for (int kc = k_start; kc <= pl; kc = next_tile(kc, KT, keep, kbeg), ++it) {
         const int buf = (VEC8 && NBUF == 2) ? (it & 1) : 0;
-        const int k0 = kc + kh * MK;                    // this group of warps' tile of the step
-        const bf16* sK = sK0 + ((size_t)buf * KT + kh * MK) * LQ;
-        const bf16* sV = sV0 + ((size_t)buf * KT + kh * MK) * MLV;
+        const int k0 = MAPS == 2 ? kc : kc + kh * MK;   // this group of warps' tile of the step
+        const bf16* sK = sK0 + ((size_t)buf * KR + kh * MK) * LQ;
+        const bf16* sV = sV0 + ((size_t)buf * KT + (MAPS == 2 ? 0 : kh * MK)) * MLV;
         if (VEC8 && NBUF == 1) {
             __syncthreads();       // every thread is done with the previous tile (and Q is staged)
             issue(kc, 0);
@@ -737,26 +807,30 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1) ? 2 : 0) attn_ch
         } else if (VEC8) {
             cp_async_wait<0>();
             __syncthreads();       // this tile has landed for every thread, and every thread is done with the other buffer
-            if (kc + KT <= pl) issue(kc + KT, buf ^ 1);
+            const int kn = next_tile(kc, KT, keep, kbeg);
+            if (kn <= pl) issue(kn, buf ^ 1);
         } else {
             auto krow = [&](int r) -> const bf16* {
-                const int pj = kc + r;
-                return pj <= pl ? k_pages + (((size_t)page_table[pj / page_size] * G + g) * page_size + pj % page_size) * D : nullptr;
+                const int pj = kc + r % KT, mp = MAPS == 2 ? r / KT : 0;
+                return pj <= pl && (pj >= kbeg || pj < keep)
+                           ? k_pages + (((size_t)page_table[pj / page_size] * G + g) * page_size + pj % page_size) * ld_k + koff + mp * D : nullptr;
             };
             auto vrow = [&](int r) -> const bf16* {
                 const int pj = kc + r;
-                return pj <= pl ? v_pages + (((size_t)page_table[pj / page_size] * G + g) * page_size + pj % page_size) * ld_v + c0 : nullptr;
+                return pj <= pl && (pj >= kbeg || pj < keep) ? v_pages + (((size_t)page_table[pj / page_size] * G + g) * page_size + pj % page_size) * ld_v + c0 : nullptr;
             };
             __syncthreads();
-            stage_bf16_rows(sK0, LQ, Dp, D, krow);
-            stage_bf16_rows(sV0, MLV, DVp, dvv, vrow);
+            stage_bf16_rows(sK0, KR, LQ, Dp, D, krow);
+            stage_bf16_rows(sV0, KT, MLV, DVp, dvv, vrow);
             __syncthreads();
         }
-        if (k0 > pl) continue;                          // no tile left for this group in the last step (barriers are above)
+        // no visible key for this group in this step (barriers are above)
+        if (k0 > pl || (k0 >= keep && k0 + MK <= kbeg)) continue;
+        const bf16* sQm = sQ + (size_t)(MAPS == 2 ? kh : 0) * MQ * LQ;
         float sc[8][4] = {};
         for (int ks = 0; ks < Dp; ks += 16) {
             uint32_t a[4];
-            ldmatrix_x4(a[0], a[1], a[2], a[3], sQ + (size_t)(warp * 16 + (lane & 15)) * LQ + ks + (lane >> 4) * 8);
+            ldmatrix_x4(a[0], a[1], a[2], a[3], sQm + (size_t)(warp * 16 + (lane & 15)) * LQ + ks + (lane >> 4) * 8);
 #pragma unroll
             for (int np = 0; np < 4; ++np) {
                 uint32_t b0, b1, b2, b3;
@@ -769,7 +843,7 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1) ? 2 : 0) attn_ch
         // A tile every row of the CTA sees in full (at or after the last row's chunk start, wholly before the first row)
         // skips the mask. The exponentials are exp2 of pre-scaled arguments: their error (2^-22) is far below the bf16
         // rounding of the weights that follows.
-        const bool full = k0 + MK - 1 <= pf && rows == MQ && k0 >= first_key(pl, chunk, opt.window);
+        const bool full = k0 + MK - 1 <= pf && rows == MQ && (k0 >= first_key(pl, chunk, opt.window) || k0 + MK <= opt.keep_first);
         float corr[2];
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
@@ -779,9 +853,10 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1) ? 2 : 0) attn_ch
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     float v = sc[j][2 * i + e] * scale;
+                    if (opt.softcap > 0.f) v = soft_cap_fast(v, opt.softcap, inv_cap);
                     if (!full) {
                         const int pj = k0 + j * 8 + 2 * tq + e;
-                        const bool ok = pj <= p_row[i] && pj >= lo_row[i] && r_lo + 8 * i < rows;
+                        const bool ok = pj <= p_row[i] && (pj >= lo_row[i] || pj < opt.keep_first) && r_lo + 8 * i < rows;
                         v = ok ? v : -INFINITY;
                     }
                     sc[j][2 * i + e] = v;
@@ -826,7 +901,60 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1) ? 2 : 0) attn_ch
             }
         }
     }
-    static_assert(KH == 1 || NV == 1, "two groups of warps exchange one 128-channel tile");
+    if constexpr (MAPS == 2) {
+        // the second map's normalised, weighted output goes to the first group through the tile buffers; o = a1 - lambda a2, the
+        // head's channels (all of them in this CTA) to unit rms, times the scale
+        float* xch = reinterpret_cast<float*>(smem_attn);
+        const int tix = threadIdx.x & 127;
+        float f[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            float lt = l[i];
+            lt += __shfl_xor_sync(0xffffffffu, lt, 1);
+            lt += __shfl_xor_sync(0xffffffffu, lt, 2);
+            f[i] = (kh == 1 ? opt.lambda : 1.f) / lt;
+        }
+        __syncthreads();                                // every warp is done with the Q, K and V buffers
+        if (kh == 1) {
+#pragma unroll
+            for (int nt = 0; nt < 16 * NV; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    if (nt * 8 < DVp) xch[(nt * 4 + e) * 128 + tix] = o[nt][e] * f[e >> 1];
+        }
+        __syncthreads();
+        if (kh == 1) return;
+        float ss[2] = {0.f, 0.f};
+#pragma unroll
+        for (int nt = 0; nt < 16 * NV; ++nt)
+            if (nt * 8 < DVp) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    // (columns past DV are zero in both maps: their V columns are staged as zeros)
+                    o[nt][e] = fmaf(o[nt][e], f[e >> 1], -xch[(nt * 4 + e) * 128 + tix]);
+                    ss[e >> 1] = fmaf(o[nt][e], o[nt][e], ss[e >> 1]);
+                }
+            }
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], 1);
+            ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], 2);
+            const int r = r_lo + 8 * i, t = t0 + r;
+            if (r >= rows) continue;
+            const float rn = opt.diff_scale / sqrtf(ss[i] / (float)DV + opt.eps);
+            bf16* orow = out + (size_t)t * ld_out + (size_t)h * DV;
+            const bool pair = (DV % 2) == 0 && ((uintptr_t)out % 4) == 0 && (ld_out % 2) == 0;
+#pragma unroll
+            for (int nt = 0; nt < 16 * NV; ++nt) {
+                const int col = nt * 8 + 2 * tq;
+                const float v0 = o[nt][2 * i] * rn, v1 = o[nt][2 * i + 1] * rn;
+                if (pair) { if (col < DV) *reinterpret_cast<uint32_t*>(orow + col) = pack_bf16x2(v0, v1); }
+                else { if (col < DV) stf(orow + col, v0); if (col + 1 < DV) stf(orow + col + 1, v1); }
+            }
+        }
+        return;
+    }
+    static_assert(KH == 1 || NV == 1 || MAPS == 2, "two groups of warps exchange one 128-channel tile");
     if (KH > 1 && NV == 1) {
         // the second group hands its (max, partial sum, unnormalised output) to the first through the tile buffers (K and V
         // buffers are contiguous; every asynchronous copy was waited for in the last step)
@@ -871,7 +999,9 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1) ? 2 : 0) attn_ch
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int col = nt * 8 + 2 * tq + e;
-                if (col < dvv) {
+                if (col < dvv && opt.raw) {
+                    opt.raw[((size_t)t * Hq + h) * DV + c0 + col] = o[nt][2 * i + e] * f;
+                } else if (col < dvv) {
                     const float gv = (gate && opt.gate_channel) ? gate_of(gate, ld_gate, t, h, c0 + col, DV, true) : 1.f;
                     stf(out + (size_t)t * ld_out + (size_t)h * DV + c0 + col, o[nt][2 * i + e] * f * gv);
                 }
@@ -915,6 +1045,57 @@ int launch_attn_mma(const float* q, const void* k_pages, const void* v_pages, co
     return cudaGetLastError() == cudaSuccess ? 0 : -100;
 }
 
+// Both maps of a head in one CTA (values of up to 256 channels). Hq counts heads, D is a map's width.
+int launch_attn_mma_maps(const float* q, const void* k_pages, const void* v_pages, const int* page_table, int page_size, void* out,
+                         int ld_out, int S, int Hq, int G, int D, int DV, int chunk, float scale, SeqPos pos, cudaStream_t s,
+                         const float* sink, int ld_v, AttnOpts opt) {
+    static SmemAttrOnce o1, o2b, o2, o1n, o2n;
+    const int Dp = (D + 15) / 16 * 16, NV = DV > 128 ? 2 : 1;
+    const bool vec8 = (D % 8) == 0 && (DV % 8) == 0 && (ld_v % 8) == 0 && ((uintptr_t)k_pages % 16) == 0 && ((uintptr_t)v_pages % 16) == 0;
+    // wide values: one CTA per SM (the accumulators fill the register file), so the next tile's copies fly while this one is
+    // computed; narrow values: one buffer and two CTAs per SM
+    const int nbuf = (vec8 && NV == 2 && Dp <= 128) ? 2 : 1;
+    auto bytes = [&](int dp) {
+        const size_t tiles = ((size_t)2 * MQ * (dp + 8) + (size_t)nbuf * MK * (2 * (dp + 8) + 128 * NV + 8)) * sizeof(bf16);
+        return std::max(tiles, (size_t)64 * NV * 128 * sizeof(float));   // the exchange of the second map's output lies over the tiles
+    };
+    const size_t smem = bytes(Dp), smem_max = bytes(nbuf == 2 ? 128 : kAttnMmaMaxDim);
+    dim3 grid(Hq, (S + MQ - 1) / MQ, 1);
+    count_launch();
+#define LCC_ATTN_MAPS(ONCE, VEC, NVN, NB)                                                                                        \
+    do {                                                                                                                         \
+        if (ensure_dyn_smem(ONCE, attn_chunk_sink_mma_kernel<VEC, 2, NVN, NB, 2>, (int)smem_max)) return -100;                   \
+        attn_chunk_sink_mma_kernel<VEC, 2, NVN, NB, 2><<<grid, 256, smem, s>>>(q, (const bf16*)k_pages, (const bf16*)v_pages, page_table, page_size, \
+                                                                               nullptr, 0, (bf16*)out, ld_out, S, Hq, G, D, DV, chunk, scale, pos, \
+                                                                               sink, ld_v, opt);                                 \
+    } while (0)
+    if (vec8 && NV == 1) LCC_ATTN_MAPS(o1, true, 1, 1);
+    else if (vec8 && nbuf == 2) LCC_ATTN_MAPS(o2b, true, 2, 2);
+    else if (vec8) LCC_ATTN_MAPS(o2, true, 2, 1);
+    else if (NV == 1) LCC_ATTN_MAPS(o1n, false, 1, 1);
+    else LCC_ATTN_MAPS(o2n, false, 2, 1);
+#undef LCC_ATTN_MAPS
+    return cudaGetLastError() == cudaSuccess ? 0 : -100;
+}
+
+// out[t, h, :] = rms(a[t, h, 0, :] - lambda * a[t, h, 1, :]) * scale (a: fp32 [S, heads, 2, DV]): the difference of two attention maps that
+// other kernels left in fp32. One warp per (row, head).
+template <typename T>
+__global__ void __launch_bounds__(128) diff_combine_kernel(const float* __restrict__ a, T* __restrict__ out, int ld_out, int S, int H, int DV,
+                                                           float lambda, float scale, float eps, SeqPos pos) {
+    if (seq_done(pos)) return;
+    const int64_t wid = (int64_t)blockIdx.x * 4 + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    if (wid >= (int64_t)S * H) return;
+    const int t = (int)(wid / H), h = (int)(wid % H);
+    const float* a1 = a + (size_t)wid * 2 * DV;
+    const float* a2 = a1 + DV;
+    float ss = 0.f;
+    for (int c = lane; c < DV; c += 32) { const float v = fmaf(-lambda, a2[c], a1[c]); ss = fmaf(v, v, ss); }
+    const float rn = scale / sqrtf(warp_sum(ss) / (float)DV + eps);
+    for (int c = lane; c < DV; c += 32) stf(out + (size_t)t * ld_out + (size_t)h * DV + c, fmaf(-lambda, a2[c], a1[c]) * rn);
+}
+
 }  // namespace
 
 int qk_norm_kv_append(int dt, const void* proj, int ld, const float* qn_w, const float* kn_w, float eps, float* q_out,
@@ -942,7 +1123,7 @@ int attn_chunk_sink(int dt, const float* q, const void* k_pages, const void* v_p
                     int DV, int chunk, float scale, bool tensor_cores, SeqPos pos, cudaStream_t s, const float* sink, int ld_v,
                     float* split_ws, size_t split_ws_floats, int key_hint) {
     return attn_masked(dt, q, k_pages, v_pages, page_table, page_size, gate, ld_gate, out, ld_out, S, Hq, G, D, DV, chunk, scale,
-                       tensor_cores, pos, s, AttnOpts{0, false, false}, sink, ld_v, split_ws, split_ws_floats, key_hint);
+                       tensor_cores, pos, s, AttnOpts{}, sink, ld_v, split_ws, split_ws_floats, key_hint);
 }
 
 int qk_headnorm_rope_append(int dt, const void* proj, int ld, int v_col, const float* qn_w, const float* kn_w, float eps,
@@ -979,12 +1160,20 @@ int attn_masked(int dt, const float* q, const void* k_pages, const void* v_pages
         return -2;
     if (ld_v <= 0) ld_v = DV;
     if (ld_v < DV) return -2;
+    if (opt.maps != 1 && (opt.maps != 2 || gate || !opt.raw)) return -2;
+    if (opt.maps == 1 && opt.raw) return -2;
     const int window = opt.window > 0 ? opt.window : 0;
+    if (opt.keep_first < 0 || (opt.keep_first > 0 && chunk > 0)) return -2;
+    const int keep = window ? opt.keep_first : 0;      // (without a window every position stays anyway)
+    AttnOpts o = opt;
+    o.keep_first = keep;
+    const int heads = Hq;
+    Hq *= opt.maps;                                    // the per-map kernels count the maps as heads
     // few rows without chunks over a long or device-known range of keys: key splits across CTAs
     int keys_est = pos.kv_len ? std::max(key_hint, pos.past + S) : pos.past + S;
-    if (window) keys_est = std::min(keys_est, window + kSplitKeys);   // the window, plus the masked head of its first tile
+    if (window) keys_est = std::min(keys_est, window + keep);
     if (chunk <= 0 && S < kAttnTiledMin && split_ws && DV <= 128 * kSplitMaxOut && Hq <= kSplitMaxHeads &&
-        ((pos.kv_len && !window) || keys_est > 2 * kSplitKeys)) {
+        ((pos.kv_len && !window) || keys_est > 2 * kSplitKeys || opt.maps == 2)) {
         const size_t per = (size_t)S * Hq * (DV + 2), cnt = kSplitCounters;
         int nz = std::min(32, std::max(1, (keys_est + kSplitKeys - 1) / kSplitKeys));
         if (split_ws_floats > cnt) nz = (int)std::min<size_t>(nz, (split_ws_floats - cnt) / per);
@@ -996,7 +1185,7 @@ int attn_masked(int dt, const float* q, const void* k_pages, const void* v_pages
             count_launch();
 #define LCC_SPLIT(T, VECB)                                                                                                   \
     attn_split_kernel<T, VECB><<<grid, 128, smem, s>>>(q, (const T*)k_pages, (const T*)v_pages, page_table, page_size, (const T*)gate,  \
-                                                       ld_gate, (T*)out, ld_out, S, Hq, G, D, DV, scale, pos, sink, ld_v, part, counters, opt)
+                                                       ld_gate, (T*)out, ld_out, S, Hq, G, D, DV, scale, pos, sink, ld_v, part, counters, o)
             if (smem > 48 * 1024) return -3;
             if (dt == DT_F32) {
                 if (((D | DV | ld_v) % 4) == 0 && (((uintptr_t)k_pages | (uintptr_t)v_pages) % 16) == 0) LCC_SPLIT(float, true); else LCC_SPLIT(float, false);
@@ -1007,24 +1196,38 @@ int attn_masked(int dt, const float* q, const void* k_pages, const void* v_pages
             return cudaGetLastError() == cudaSuccess ? 0 : -100;
         }
     }
+    // the maps of a differential layer that the kernels below leave in fp32
+    auto combine = [&]() -> int {
+        if (opt.maps == 1) return 0;
+        const int blocks = (int)(((int64_t)S * heads + 3) / 4);
+        count_launch();
+        if (dt == DT_F32)
+            diff_combine_kernel<float><<<blocks, 128, 0, s>>>(opt.raw, (float*)out, ld_out, S, heads, DV, opt.lambda, opt.diff_scale, opt.eps, pos);
+        else
+            diff_combine_kernel<bf16><<<blocks, 128, 0, s>>>(opt.raw, (bf16*)out, ld_out, S, heads, DV, opt.lambda, opt.diff_scale, opt.eps, pos);
+        return cudaGetLastError() == cudaSuccess ? 0 : -100;
+    };
     // The one-CTA-per-row kernel keeps one score per key of the longest range a row of this call can see in shared memory
     // (a chunk, a window, or everything cached when the host knows the length). Ranges that do not fit (or whose length only
     // the device knows, in a replayed step without chunks or window) go to the tiled kernels, which walk the keys in tiles
     // and take any row count.
     int max_keys = chunk > 0 ? chunk : -1;
-    if (window) max_keys = max_keys > 0 ? std::min(max_keys, window) : window;
+    if (window) max_keys = max_keys > 0 ? std::min(max_keys, window) : window + keep;
     if (!pos.kv_len) max_keys = max_keys > 0 ? std::min(max_keys, pos.past + S) : pos.past + S;
     const size_t smem = sizeof(float) * ((size_t)D + (size_t)std::max(max_keys, 0));
     static const bool force_tiled = [] { const char* e = getenv("LIVECC_B200_SEQ_ATTN_TILED"); return e && e[0] == '1'; }();
     if (S >= kAttnTiledMin || max_keys < 0 || smem > 160 * 1024 || force_tiled) {
-        if (dt == DT_BF16 && tensor_cores && D <= kAttnMmaMaxDim)
-            return launch_attn_mma(q, k_pages, v_pages, page_table, page_size, gate, ld_gate, out, ld_out, S, Hq, G, D, DV, chunk,
-                                   scale, pos, s, sink, ld_v, opt);
-        if (dt == DT_F32)
-            return launch_attn_tiled<float>(q, k_pages, v_pages, page_table, page_size, gate, ld_gate, out, ld_out, S, Hq, G, D, DV,
-                                            chunk, scale, pos, s, sink, ld_v, opt);
-        return launch_attn_tiled<bf16>(q, k_pages, v_pages, page_table, page_size, gate, ld_gate, out, ld_out, S, Hq, G, D, DV, chunk,
-                                       scale, pos, s, sink, ld_v, opt);
+        const bool mma = dt == DT_BF16 && tensor_cores && D <= kAttnMmaMaxDim;
+        if (mma && opt.maps == 2 && DV <= 256)
+            return launch_attn_mma_maps(q, k_pages, v_pages, page_table, page_size, out, ld_out, S, heads, G, D, DV, chunk, scale, pos, s,
+                                        sink, ld_v, o);
+        const int rc = mma ? launch_attn_mma(q, k_pages, v_pages, page_table, page_size, gate, ld_gate, out, ld_out, S, Hq, G, D, DV, chunk,
+                                             scale, pos, s, sink, ld_v, o)
+                       : dt == DT_F32 ? launch_attn_tiled<float>(q, k_pages, v_pages, page_table, page_size, gate, ld_gate, out, ld_out, S, Hq, G, D,
+                                                                 DV, chunk, scale, pos, s, sink, ld_v, o)
+                                      : launch_attn_tiled<bf16>(q, k_pages, v_pages, page_table, page_size, gate, ld_gate, out, ld_out, S, Hq, G, D,
+                                                                DV, chunk, scale, pos, s, sink, ld_v, o);
+        return rc ? rc : combine();
     }
     dim3 grid(S, Hq);
     count_launch();
@@ -1032,14 +1235,14 @@ int attn_masked(int dt, const float* q, const void* k_pages, const void* v_pages
         if (smem > 48 * 1024) cudaFuncSetAttribute(attn_chunk_sink_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         attn_chunk_sink_kernel<float><<<grid, 128, smem, s>>>(q, (const float*)k_pages, (const float*)v_pages, page_table,
                                                               page_size, (const float*)gate, ld_gate, (float*)out, ld_out, S, Hq,
-                                                              G, D, DV, chunk, scale, pos, sink, ld_v, opt);
+                                                              G, D, DV, chunk, scale, pos, sink, ld_v, o);
     } else {
         if (smem > 48 * 1024) cudaFuncSetAttribute(attn_chunk_sink_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         attn_chunk_sink_kernel<bf16><<<grid, 128, smem, s>>>(q, (const bf16*)k_pages, (const bf16*)v_pages, page_table,
                                                              page_size, (const bf16*)gate, ld_gate, (bf16*)out, ld_out, S, Hq, G,
-                                                             D, DV, chunk, scale, pos, sink, ld_v, opt);
+                                                             D, DV, chunk, scale, pos, sink, ld_v, o);
     }
-    return cudaGetLastError() == cudaSuccess ? 0 : -100;
+    return cudaGetLastError() == cudaSuccess ? combine() : -100;
 }
 
 }  // namespace lcc

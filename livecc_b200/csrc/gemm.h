@@ -21,6 +21,7 @@ enum GemmEpilogue {
     EPI_CLAMP_GLU = 10,      // gate/up rows interleaved by 16 as for EPI_SWIGLU: g = min(gate, limit), u = clamp(up, +-limit),
                              // C[:, j] = bf16(g * sigmoid(alpha g) * (u + up_bias)) in fp32 on the accumulators; limit = epi_param,
                              // alpha = epi_alpha, up_bias = epi_up_bias (1, 0 and an infinite limit: silu(gate) * up)
+    EPI_GELU_ERF = 11,       // C = bf16(gelu_erf(acc)), the activation in fp32 on the accumulator
 };
 
 struct GemmArgs {

@@ -35,7 +35,7 @@ __device__ __forceinline__ float y_value(const YSource<T>& s, int r, int c) {
     float acc = 0.f;
     for (int k = 0; k < s.top; ++k)
         acc = fmaf(s.weight[(size_t)r * s.top + k], ldf(s.eo + (size_t)s.pos[(size_t)r * s.top + k] * s.ld_eo + c), acc);
-    if (s.so) acc = fmaf(s.gate[r], ldf(s.so + (size_t)r * s.ld_so + c), acc);
+    if (s.so) acc = fmaf((s.gate ? s.gate[r] : 1.f), ldf(s.so + (size_t)r * s.ld_so + c), acc);
     return acc;
 }
 
@@ -68,7 +68,7 @@ __global__ void __launch_bounds__(256) hyper_boundary_kernel(float* __restrict__
         int pk[kMaxTop];
         float wk[kMaxTop];
         const bool routed = !src.y && src.eo;
-        const float gs = (routed && src.so) ? src.gate[r] : 0.f;
+        const float gs = (routed && src.so) ? (src.gate ? src.gate[r] : 1.f) : 0.f;
         if (routed) {
 #pragma unroll
             for (int k = 0; k < kMaxTop; ++k) {
@@ -206,7 +206,7 @@ int hyper_boundary(int dt, float* xs, int n, const void* y, int ld_y, const floa
                    float eps, void* xa, float* sum_out, int S, int W, cudaStream_t s, const MoeCombine* mc) {
     const bool has_y = y || mc;
     if (!xs || n < 1 || n > kMaxStreams || S < 1 || W < 1 || (has_y && !prev) || (w && (!next || !xa)) || (y && mc)) return -2;
-    if (mc && (!mc->eo || !mc->pos || !mc->weight || mc->top < 1 || (mc->so && !mc->gate))) return -2;
+    if (mc && (!mc->eo || !mc->pos || !mc->weight || mc->top < 1)) return -2;
     if (!has_y && !w && !sum_out) return 0;
     if (dt == DT_F32) {
         YSource<float> src{(const float*)y, ld_y, nullptr, 0, nullptr, nullptr, 0, nullptr, 0, nullptr};

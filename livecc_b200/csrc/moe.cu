@@ -25,7 +25,7 @@ __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-
 constexpr int kMaxExpertsPerLane = 16;   // experts <= 512
 // The choice for one row by one warp; lane 0 returns the k-th expert and its score through `emit`.
 // ro.softmax: score = softmax over the E outputs (else a sigmoid each). ro.groups > 0: the outputs form equal groups of
-// neighbours; a group scores as its largest choice score, the ro.keep best groups stay (ties: the lower index) and every
+// neighbours; a group scores as its largest choice score (ro.group_top = 2: the sum of its two largest), the ro.keep best groups stay (ties: the lower index) and every
 // other output's choice score counts as -inf. gch / gkeep: this warp's scratch in shared memory ([E] floats, [groups] flags).
 template <typename Emit>
 __device__ __forceinline__ void route_row(const float* __restrict__ z, const float* __restrict__ correction, int E, int top,
@@ -66,8 +66,12 @@ __device__ __forceinline__ void route_row(const float* __restrict__ z, const flo
             int bg = 0x7fffffff;
             for (int g = lane; g < ro.groups; g += 32) {
                 if (gkeep[g]) continue;
-                float m = -INFINITY;
-                for (int j = 0; j < per; ++j) m = fmaxf(m, gch[g * per + j]);
+                float m = -INFINITY, m2 = -INFINITY;      // the group's largest and second largest choice score
+                for (int j = 0; j < per; ++j) {
+                    const float c = gch[g * per + j];
+                    if (c > m) { m2 = m; m = c; } else m2 = fmaxf(m2, c);
+                }
+                if (ro.group_top == 2 && per > 1) m += m2;
                 if (m > best || bg == 0x7fffffff) { best = m; bg = g; }   // ascending g: the first of equals stays
             }
 #pragma unroll
@@ -235,7 +239,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ eo, int ld_eo, const in
             const int p = pos[(size_t)r * top + k];
             if (p >= 0) acc = fmaf(weight[(size_t)r * top + k], ldf(eo + (size_t)p * ld_eo + c), acc);
         }
-        if (so) acc = fmaf(shared_gate[r], ldf(so + (size_t)r * ld_so + c), acc);
+        if (so) acc = fmaf(shared_gate ? shared_gate[r] : 1.f, ldf(so + (size_t)r * ld_so + c), acc);
         stf(out + (size_t)r * ld_out + c, acc);
     }
 }
@@ -246,6 +250,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ eo, int ld_eo, const in
 static bool router_ok(const MoeRouterOpts& ro, int E, int top, const float* shared_gate) {
     if (ro.identity < 0 || ro.identity >= E || (ro.identity > 0 && !shared_gate)) return false;
     if (ro.groups > 0 && (E % ro.groups || ro.keep < 1 || ro.keep > ro.groups || ro.keep * (E / ro.groups) < top)) return false;
+    if (ro.group_top < 1 || ro.group_top > 2) return false;
     if (ro.topk_softmax && (ro.identity > 0 || ro.groups > 0 || ro.softmax)) return false;
     return ro.groups >= 0;
 }
@@ -295,7 +300,7 @@ int moe_gather_rows(int dt, const void* in, int ld_in, const int* src_row, void*
 
 int moe_combine(int dt, const void* eo, int ld_eo, const int* pos, const float* weight, int top, const void* so, int ld_so,
                 const float* shared_gate, void* out, int ld_out, int S, int W, cudaStream_t s) {
-    if (!eo || !pos || !weight || !out || S < 1 || W < 1 || top < 1 || (so && !shared_gate)) return -2;
+    if (!eo || !pos || !weight || !out || S < 1 || W < 1 || top < 1) return -2;
     count_launch();
     if (dt == DT_F32)
         moe_combine_kernel<float><<<S, 256, 0, s>>>((const float*)eo, ld_eo, pos, weight, top, (const float*)so, ld_so, shared_gate,

@@ -37,11 +37,13 @@ __global__ void __launch_bounds__(256) rotary_pack_kernel(const T* __restrict__ 
             const int d = i % sg.dim, hb = i - d;
             const int r = d - sg.rot_off;
             float v = ldf(row + sg.col_in + i);
+            if (sg.silu) v = v / (1.f + expf(-v));
             if (r >= 0 && r < sg.rot_dims) {
                 const int j = r < half ? r : r - half;
                 const float ang = p * inv_freq[j];
                 const float c = cosf(ang) * mag, s = sinf(ang) * mag;
-                const float other = ldf(row + sg.col_in + hb + sg.rot_off + (r < half ? r + half : r - half));
+                float other = ldf(row + sg.col_in + hb + sg.rot_off + (r < half ? r + half : r - half));
+                if (sg.silu) other = other / (1.f + expf(-other));
                 v = r < half ? v * c - other * s : v * c + other * s;
             }
             orow[sg.col_out + i] = v * sg.scale;

@@ -237,14 +237,18 @@ __global__ void __launch_bounds__(256) gather_norm_kernel(const float* __restric
     __shared__ float red[32];
     const int i = blockIdx.x;
     const float* x = x32 + (size_t)rows[i] * W;
-    float rn = 1.f;
-    if (n.kind == NORM_RMS) {
+    float rn = 1.f, mean = 0.f;
+    if (n.kind != NORM_DYT) {
         float ss = 0.f;
-        for (int c = threadIdx.x; c < W; c += blockDim.x) ss = fmaf(x[c], x[c], ss);
+        if (n.kind == NORM_LAYER) {
+            for (int c = threadIdx.x; c < W; c += blockDim.x) mean += x[c];
+            mean = block_sum(mean, red) / (float)W;
+        }
+        for (int c = threadIdx.x; c < W; c += blockDim.x) ss = fmaf(x[c] - mean, x[c] - mean, ss);
         ss = block_sum(ss, red);
         rn = 1.f / sqrtf(ss / (float)W + n.eps);
     }
-    for (int c = threadIdx.x; c < W; c += blockDim.x) stf(out + (size_t)i * W + c, norm_apply(n, x[c], rn, c));
+    for (int c = threadIdx.x; c < W; c += blockDim.x) stf(out + (size_t)i * W + c, norm_apply(n, x[c] - mean, rn, c));
 }
 
 template <typename T> __device__ __forceinline__ void ld4(const T* p, float (&v)[4]);
@@ -292,7 +296,7 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(float* __restrict__ 
             }
             __syncthreads();
         }
-        const float gs = (has_mc && mc.so) ? mc.gate[r] : 0.f;
+        const float gs = (has_mc && mc.so) ? (mc.gate ? mc.gate[r] : 1.f) : 0.f;
         for (int c = threadIdx.x * V; c < W; c += blockDim.x * V) {
             float y[V], t[V];
 #pragma unroll
@@ -326,16 +330,22 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(float* __restrict__ 
             float v[V];
             if (VEC) ld4(x + c, (float(&)[4])v); else v[0] = x[c];
 #pragma unroll
-            for (int i = 0; i < V; ++i) { v[i] += y[i]; ss = fmaf(v[i], v[i], ss); }
+            for (int i = 0; i < V; ++i) { v[i] += y[i]; ss = n.kind == NORM_LAYER ? ss + v[i] : fmaf(v[i], v[i], ss); }
             if (VEC) st4(x + c, (const float(&)[4])v); else x[c] = v[0];
         }
-    } else if (n.w && n.kind == NORM_RMS) {
-        for (int c = threadIdx.x; c < W; c += blockDim.x) ss = fmaf(x[c], x[c], ss);
+    } else if (n.w && n.kind != NORM_DYT) {
+        for (int c = threadIdx.x; c < W; c += blockDim.x) ss = n.kind == NORM_LAYER ? ss + x[c] : fmaf(x[c], x[c], ss);
     }
     if (!n.w) return;
-    float rn = 1.f;
-    if (n.kind == NORM_RMS) {
+    float rn = 1.f, mean = 0.f;
+    if (n.kind != NORM_DYT) {
         ss = block_sum(ss, red);
+        if (n.kind == NORM_LAYER) {        // ss is the row's sum: the squared deviations take a pass of their own
+            mean = ss / (float)W;
+            ss = 0.f;
+            for (int c = threadIdx.x; c < W; c += blockDim.x) ss = fmaf(x[c] - mean, x[c] - mean, ss);   // (pass 1 ended in a barrier: block_sum)
+            ss = block_sum(ss, red);
+        }
         rn = 1.f / sqrtf(ss / (float)W + n.eps);
     }
     // (a thread rewrites in xa only the columns it read in pass 1: an xa row that served as an addend is safe)
@@ -343,7 +353,7 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(float* __restrict__ 
         float v[V];
         if (VEC) ld4(x + c, (float(&)[4])v); else v[0] = x[c];
 #pragma unroll
-        for (int i = 0; i < V; ++i) v[i] = norm_apply(n, v[i], rn, c + i);
+        for (int i = 0; i < V; ++i) v[i] = norm_apply(n, v[i] - mean, rn, c + i);
         if (VEC) st4(xa + (size_t)r * W + c, (const float(&)[4])v); else stf(xa + (size_t)r * W + c, v[0]);
     }
 }
@@ -383,7 +393,7 @@ __global__ void __launch_bounds__(256) branch_norm_residual_kernel(float* __rest
         }
         __syncthreads();
     }
-    const float gs = (has_mc && mc.so) ? mc.gate[r] : 0.f;
+    const float gs = (has_mc && mc.so) ? (mc.gate ? mc.gate[r] : 1.f) : 0.f;
     auto value = [&](int c, float (&y)[V]) {
         float t[V];
         if (!has_mc) {
@@ -452,6 +462,134 @@ __global__ void __launch_bounds__(256) branch_norm_residual_kernel(float* __rest
             update(c, y, rn);
         }
     }
+}
+
+// A norm on either side of a sublayer, one CTA per row: the sublayer's row y (or the routed feed-forward's weighted sum) is
+// normed and added to the fp32 residual row, and the new row is normed for the next sublayer. y and the new row stay in registers
+// between their statistics and their use (E pieces of V columns per thread; E = 0: rows wider than 256 * 16 pieces form y again in
+// every pass and read the residual row back). A layer norm's variance is the mean of the squared deviations from the mean that a first
+// reduction gave. A column's sums run in the same order for every S.
+template <typename T, int E, bool VEC>
+__global__ void __launch_bounds__(256) sandwich_residual_kernel(float* __restrict__ x32, const T* __restrict__ a, int ld_a, bool has_mc,
+                                                                MoeCombine mc, NormSpec post, NormSpec next, T* __restrict__ xa, int W) {
+    __shared__ float red[32];
+    __shared__ int spos[kCombineTop];
+    __shared__ float swt[kCombineTop];
+    constexpr int V = VEC ? 4 : 1;
+    constexpr int EN = E > 0 ? E : 1;
+    const int r = blockIdx.x;
+    float* x = x32 + (size_t)r * W;
+    const int top = has_mc ? mc.top : 0;
+    const bool cached = top <= kCombineTop;
+    const float inv_w = 1.f / (float)W;
+    float vx[EN][V], vy[EN][V];
+    if (E > 0) {            // the residual row's loads fly while y is formed and reduced
+#pragma unroll
+        for (int i = 0; i < EN; ++i) {
+            const int c = (threadIdx.x + i * 256) * V;
+#pragma unroll
+            for (int u = 0; u < V; ++u) vx[i][u] = vy[i][u] = 0.f;
+            if (c < W) { if (VEC) ld4(x + c, (float(&)[4])vx[i]); else vx[i][0] = x[c]; }
+        }
+    }
+    if (has_mc && cached) {
+        if (threadIdx.x < top) {
+            spos[threadIdx.x] = mc.pos[(size_t)r * top + threadIdx.x];
+            swt[threadIdx.x] = mc.weight[(size_t)r * top + threadIdx.x];
+        }
+        __syncthreads();
+    }
+    const float gs = (has_mc && mc.so) ? (mc.gate ? mc.gate[r] : 1.f) : 0.f;
+    auto value = [&](int c, float (&y)[V]) {
+        float t[V];
+        if (!has_mc) {
+            if (VEC) ld4(a + (size_t)r * ld_a + c, (float(&)[4])y); else y[0] = ldf(a + (size_t)r * ld_a + c);
+            return;
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) y[i] = 0.f;
+        for (int k = 0; k < top; ++k) {
+            const int p = cached ? spos[k] : mc.pos[(size_t)r * top + k];
+            if (p < 0) continue;
+            const float wk = cached ? swt[k] : mc.weight[(size_t)r * top + k];
+            const T* src = (const T*)mc.eo + (size_t)p * mc.ld_eo + c;
+            if (VEC) ld4(src, (float(&)[4])t); else t[0] = ldf(src);
+#pragma unroll
+            for (int i = 0; i < V; ++i) y[i] = fmaf(wk, t[i], y[i]);
+        }
+        if (mc.so) {
+            const T* src = (const T*)mc.so + (size_t)r * mc.ld_so + c;
+            if (VEC) ld4(src, (float(&)[4])t); else t[0] = ldf(src);
+#pragma unroll
+            for (int i = 0; i < V; ++i) y[i] = fmaf(gs, t[i], y[i]);
+        }
+    };
+    // visit(c, y, i): every piece of this thread, y in registers or formed again
+    auto each_y = [&](auto visit) {
+        if (E > 0) {
+#pragma unroll
+            for (int i = 0; i < EN; ++i) { const int c = (threadIdx.x + i * 256) * V; if (c < W) visit(c, vy[i], vx[i]); }
+        } else {
+            for (int c = threadIdx.x * V; c < W; c += 256 * V) {
+                float y[V], xv[V];
+                value(c, y);
+                if (VEC) ld4(x + c, (float(&)[4])xv); else xv[0] = x[c];
+                visit(c, y, xv);
+            }
+        }
+    };
+    auto each_x = [&](auto visit) {
+        if (E > 0) {
+#pragma unroll
+            for (int i = 0; i < EN; ++i) { const int c = (threadIdx.x + i * 256) * V; if (c < W) visit(c, vx[i]); }
+        } else {
+            for (int c = threadIdx.x * V; c < W; c += 256 * V) {
+                float xv[V];
+                if (VEC) ld4(x + c, (float(&)[4])xv); else xv[0] = x[c];
+                visit(c, xv);
+            }
+        }
+    };
+    if (E > 0) {
+#pragma unroll
+        for (int i = 0; i < EN; ++i) { const int c = (threadIdx.x + i * 256) * V; if (c < W) value(c, vy[i]); }
+    }
+    float mean = 0.f, ss = 0.f;
+    if (post.kind == NORM_LAYER) {
+        each_y([&](int, const float (&y)[V], const float (&)[V]) {
+#pragma unroll
+            for (int u = 0; u < V; ++u) mean += y[u];
+        });
+        mean = block_sum(mean, red) * inv_w;
+    }
+    each_y([&](int, const float (&y)[V], const float (&)[V]) {
+#pragma unroll
+        for (int u = 0; u < V; ++u) ss = fmaf(y[u] - mean, y[u] - mean, ss);
+    });
+    float rn = 1.f / sqrtf(block_sum(ss, red) * inv_w + post.eps);
+    float sum = 0.f;
+    each_y([&](int c, const float (&y)[V], float (&xv)[V]) {
+        float w[V];
+        if (VEC) ld4(post.w + c, (float(&)[4])w); else w[0] = post.w[c];
+#pragma unroll
+        for (int u = 0; u < V; ++u) { xv[u] = fmaf((y[u] - mean) * rn, w[u], xv[u]); sum += xv[u]; }
+        if (VEC) st4(x + c, (const float(&)[4])xv); else x[c] = xv[0];
+    });
+    if (!next.w) return;
+    mean = 0.f; ss = 0.f;
+    if (next.kind == NORM_LAYER) mean = block_sum(sum, red) * inv_w;
+    each_x([&](int, const float (&xv)[V]) {
+#pragma unroll
+        for (int u = 0; u < V; ++u) ss = fmaf(xv[u] - mean, xv[u] - mean, ss);
+    });
+    rn = 1.f / sqrtf(block_sum(ss, red) * inv_w + next.eps);
+    each_x([&](int c, const float (&xv)[V]) {
+        float w[V], v[V];
+        if (VEC) ld4(next.w + c, (float(&)[4])w); else w[0] = next.w[c];
+#pragma unroll
+        for (int u = 0; u < V; ++u) v[u] = (xv[u] - mean) * rn * w[u];
+        if (VEC) st4(xa + (size_t)r * W + c, (const float(&)[4])v); else stf(xa + (size_t)r * W + c, v[0]);
+    });
 }
 
 inline int done() { return cudaGetLastError() == cudaSuccess ? 0 : -100; }
@@ -561,7 +699,7 @@ int softcap(float* x, int64_t n, float cap, cudaStream_t s, float scale) {
 }
 
 int gather_norm(int dt, const float* x32, const int* rows, const NormSpec& n, void* out, int n_rows, int W, cudaStream_t s) {
-    if (!x32 || !rows || !n.w || !out || n_rows < 1 || W < 1 || (n.kind == NORM_DYT && !n.b) || (n.kind != NORM_DYT && n.kind != NORM_RMS))
+    if (!x32 || !rows || !n.w || !out || n_rows < 1 || W < 1 || (n.kind == NORM_DYT && !n.b) || (n.kind != NORM_DYT && n.kind != NORM_RMS && n.kind != NORM_LAYER))
         return -2;
     count_launch();
     if (dt == DT_F32)
@@ -574,9 +712,9 @@ int gather_norm(int dt, const float* x32, const int* rows, const NormSpec& n, vo
 int residual_norm(int dt, float* x32, const void* a, int ld_a, const void* b, int ld_b, const MoeCombine* mc, const NormSpec& next,
                   void* xa, int S, int W, cudaStream_t s) {
     if (!x32 || S < 1 || W < 1 || (next.w && !xa) || (next.w && next.kind == NORM_DYT && !next.b) ||
-        (next.kind != NORM_DYT && next.kind != NORM_RMS) || (mc && b))
+        (next.kind != NORM_DYT && next.kind != NORM_RMS && next.kind != NORM_LAYER) || (mc && b))
         return -2;
-    if (mc && (!mc->eo || !mc->pos || !mc->weight || mc->top < 1 || (mc->so && !mc->gate))) return -2;
+    if (mc && (!mc->eo || !mc->pos || !mc->weight || mc->top < 1)) return -2;
     if (!a && !b && !mc && !next.w) return 0;
     count_launch();
     const MoeCombine m = mc ? *mc : MoeCombine{};
@@ -595,7 +733,7 @@ int residual_norm(int dt, float* x32, const void* a, int ld_a, const void* b, in
 int branch_norm_residual(int dt, float* x32, const void* a, int ld_a, const MoeCombine* mc, const float* w, float eps, void* xa,
                          int S, int W, cudaStream_t s) {
     if (!x32 || !w || S < 1 || W < 1 || (!a && !mc) || (a && mc)) return -2;
-    if (mc && (!mc->eo || !mc->pos || !mc->weight || mc->top < 1 || (mc->so && !mc->gate))) return -2;
+    if (mc && (!mc->eo || !mc->pos || !mc->weight || mc->top < 1)) return -2;
     count_launch();
     const MoeCombine m = mc ? *mc : MoeCombine{};
     const size_t es = dt == DT_F32 ? 4 : 2;
@@ -617,6 +755,35 @@ int branch_norm_residual(int dt, float* x32, const void* a, int ld_a, const MoeC
     else LCC_BNR(0);
 #undef LCC_BNR
 #undef LCC_BNR2
+    return done();
+}
+
+int sandwich_residual(int dt, float* x32, const void* a, int ld_a, const MoeCombine* mc, const NormSpec& post, const NormSpec& next, void* xa,
+                      int S, int W, cudaStream_t s) {
+    auto kind_ok = [](int k) { return k == NORM_RMS || k == NORM_LAYER; };
+    if (!x32 || !post.w || S < 1 || W < 1 || (!a && !mc) || (a && mc) || (next.w && !xa) || !kind_ok(post.kind) || !kind_ok(next.kind)) return -2;
+    if (mc && (!mc->eo || !mc->pos || !mc->weight || mc->top < 1)) return -2;
+    count_launch();
+    const MoeCombine m = mc ? *mc : MoeCombine{};
+    const size_t es = dt == DT_F32 ? 4 : 2;
+    auto ok4 = [&](const void* p, int ld) { return !p || ((ld % 4) == 0 && ((uintptr_t)p % (4 * es)) == 0); };
+    const bool vec = (W % 4) == 0 && ((uintptr_t)x32 % 16) == 0 && ((uintptr_t)post.w % 16) == 0 && ((uintptr_t)next.w % 16) == 0 && ok4(a, ld_a) &&
+                     ok4(xa, W) && (!mc || (ok4(m.eo, m.ld_eo) && ok4(m.so, m.ld_so)));
+#define LCC_SR2(E, VECB)                                                                                                       \
+    do {                                                                                                                       \
+        if (dt == DT_F32) sandwich_residual_kernel<float, E, VECB><<<S, 256, 0, s>>>(x32, (const float*)a, ld_a, mc != nullptr, m, post, next, (float*)xa, W); \
+        else sandwich_residual_kernel<bf16, E, VECB><<<S, 256, 0, s>>>(x32, (const bf16*)a, ld_a, mc != nullptr, m, post, next, (bf16*)xa, W);                 \
+    } while (0)
+#define LCC_SR(E) do { if (vec) LCC_SR2(E, true); else LCC_SR2(E, false); } while (0)
+    const int per = (W / (vec ? 4 : 1) + 255) / 256;      // pieces per thread: the form depends on the row's width alone
+    if (per <= 1) LCC_SR(1);
+    else if (per <= 2) LCC_SR(2);
+    else if (per <= 4) LCC_SR(4);
+    else if (per <= 8) LCC_SR(8);
+    else if (per <= kRowCache) LCC_SR(16);
+    else LCC_SR(0);
+#undef LCC_SR
+#undef LCC_SR2
     return done();
 }
 

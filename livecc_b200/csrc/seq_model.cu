@@ -3,8 +3,8 @@
 // same launch sequence; what differs is the row count and which kernel of an op the shape selects.
 // A layer is a mixer (its output lands in one buffer), a feed-forward (dense or routed) and the block form around them
 // (post-norm residual, pre-norm sublayers on several residual streams, a parallel block whose mixer and feed-forward read
-// one normed row, or sublayers that read the residual stream itself and are normed on their way back into it); the three are
-// chosen independently per model.
+// one normed row, sublayers that read the residual stream itself and are normed on their way back into it, or sublayers with a
+// norm on either side); the three are chosen independently per model.
 // The host (Python) owns every buffer; this file only sequences kernel launches.
 #include <stdlib.h>
 #include <string.h>
@@ -76,7 +76,8 @@ Dims dims_of(const lcc_seq_layer& L) {
         z.a_lat = L.a_heads * L.a_rank;
         z.a_o = L.a_heads * L.a_vdim;
     } else if (L.type == LCC_MIX_ATTENTION) {
-        z.m_nq = L.m_heads * L.m_dim; z.m_nk = L.m_kv_heads * L.m_dim;
+        const int maps = L.m_maps > 1 ? L.m_maps : 1;
+        z.m_nq = L.m_heads * maps * L.m_dim; z.m_nk = L.m_kv_heads * maps * L.m_dim;
         z.m_nv = L.m_value_keys ? 0 : L.m_kv_heads * L.m_vdim;
         z.m_vcol = L.m_value_keys ? z.m_nq : z.m_nq + z.m_nk;       // the values are the key columns as projected, or their own
         z.m_gate = z.m_nq + z.m_nk + z.m_nv;
@@ -150,8 +151,10 @@ WsLayout make_layout(const lcc_seq_model* m, int NT, int NW) {
             split_floats = std::max(split_floats, lcc::attn_split_ws_floats(lcc::kAttnTiledMin - 1, l.l_heads, l.l_vdim));
         if (l.type == LCC_MIX_ATTENTION) {
             wp = std::max(wp, ld8(z.m_proj)); wm = std::max(wm, ld8(z.m_o)); wq = std::max(wq, z.m_nq);
+            const int maps = l.m_maps > 1 ? l.m_maps : 1;
+            if (maps > 1) wy = std::max(wy, l.m_heads * maps * l.m_vdim);      // the maps' outputs in fp32, where no kernel takes their difference itself
             if (l.m_chunk <= 0)
-                split_floats = std::max(split_floats, lcc::attn_split_ws_floats(lcc::kAttnTiledMin - 1, l.m_heads, l.m_vdim));
+                split_floats = std::max(split_floats, lcc::attn_split_ws_floats(lcc::kAttnTiledMin - 1, l.m_heads * maps, l.m_vdim));
         }
         if (l.ff_kind == LCC_FF_MOE) {
             const bool glu = l.e_act == LCC_EXPERT_CLAMP_GLU || l.e_act == LCC_EXPERT_SILU_GLU;
@@ -221,7 +224,9 @@ int linear(const lcc_seq_model* m, const void* x, int ldx, const void* W, const 
         a.c_f32 = y_f32;
         a.A = x; a.B = W; a.C = y; a.M = M; a.N = Np; a.K = K; a.lda = ldx; a.ldb = K; a.ldc = ldy;
         a.bias = bias ? bias_st : nullptr; a.residual = nullptr; a.ldr = 0; a.block_n = 0;
-        a.epi = act == lcc::ACT_RELU2 ? lcc::EPI_RELU2 : (act == lcc::ACT_GELU_TANH ? lcc::EPI_GELU_TANH : (bias ? lcc::EPI_BIAS : lcc::EPI_NONE));
+        a.epi = act == lcc::ACT_RELU2 ? lcc::EPI_RELU2
+                : act == lcc::ACT_GELU_TANH ? lcc::EPI_GELU_TANH
+                : act == lcc::ACT_GELU_ERF ? lcc::EPI_GELU_ERF : (bias ? lcc::EPI_BIAS : lcc::EPI_NONE);
         return lcc::gemm_bf16_tn(a, m->ctx->num_sms, s);
     }
     if (act != lcc::ACT_NONE) {   // the activation rides in the store of the CUDA-core kernels too
@@ -263,13 +268,15 @@ lcc_seq_model* lcc_seq_model_create(lcc_ctx* ctx, const lcc_seq_model_desc* desc
     if (desc->width < 1 || desc->vocab < 1 || desc->n_layers < 1) return fail("bad sizes");
     if (desc->dtype != LCC_DT_BF16 && desc->dtype != LCC_DT_F32) return fail("unknown storage type");
     if (!desc->embed || !desc->final_norm_f32 || !desc->head) return fail("missing weights");
-    const bool hc = desc->block == LCC_BLOCK_PRENORM_HC, par = desc->block == LCC_BLOCK_PARALLEL, bn = desc->block == LCC_BLOCK_BRANCHNORM;
+    const bool hc = desc->block == LCC_BLOCK_PRENORM_HC, par = desc->block == LCC_BLOCK_PARALLEL, bn = desc->block == LCC_BLOCK_BRANCHNORM,
+               sw = desc->block == LCC_BLOCK_SANDWICH;
     const bool dyt = desc->norm_kind == LCC_NORM_DYT;
-    if (desc->block != LCC_BLOCK_POSTNORM && !hc && !par && !bn) return fail("unknown block form");
+    if (desc->block != LCC_BLOCK_POSTNORM && !hc && !par && !bn && !sw) return fail("unknown block form");
     if (bn && (desc->canon_taps < 0 || desc->canon_taps > 8)) return fail("at most 8 taps in the convolution in front of a mixer");
     bool vkeep_seen = false;
     int vkeep_cols = 0;
-    if (desc->norm_kind != LCC_NORM_RMS && !dyt) return fail("unknown norm kind");
+    if (desc->norm_kind != LCC_NORM_RMS && desc->norm_kind != LCC_NORM_LAYER && !dyt) return fail("unknown norm kind");
+    if (desc->norm_kind == LCC_NORM_LAYER && !sw) return fail("layer norms are served in sandwich blocks");
     if (dyt && (!par || !desc->final_norm_bias_f32)) return fail("the Dynamic-Tanh norm is served in parallel blocks and needs its bias");
     if (hc && (desc->streams < 1 || desc->streams > 8)) return fail("1 to 8 residual streams");
     for (int i = 0; i < desc->n_layers; ++i) {
@@ -277,7 +284,7 @@ lcc_seq_model* lcc_seq_model_create(lcc_ctx* ctx, const lcc_seq_model_desc* desc
         if (l.ff_kind == LCC_FF_MOE) {
             if (l.e_experts < 1 || l.e_experts > 512 || l.e_top < 1 || l.e_top > l.e_experts + std::max(l.e_identity, 0) || l.e_ff < 1 || l.e_shared_ff < 0)
                 return fail("routed feed-forward: unsupported sizes");
-            if ((!par && !l.norm2_f32) || !l.e_router || (!l.e_correction_f32 && l.e_router_kind != LCC_ROUTER_TOPK_SOFTMAX) || !l.e_up || !l.e_down || (l.e_shared_ff > 0 && (!l.e_shared_up || !l.e_shared_down)))
+            if ((!par && !l.norm2_f32) || !l.e_router || !l.e_up || !l.e_down || (l.e_shared_ff > 0 && (!l.e_shared_up || !l.e_shared_down)))
                 return fail("routed feed-forward: missing weights");
             const int outs = l.e_experts + l.e_identity;
             if (l.e_identity < 0 || outs > 512 || l.e_top > outs || (l.e_identity > 0 && (l.e_shared_ff > 0 || !par)))
@@ -287,17 +294,20 @@ lcc_seq_model* lcc_seq_model_create(lcc_ctx* ctx, const lcc_seq_model_desc* desc
             if (l.e_router_kind != LCC_ROUTER_SIGMOID && l.e_router_kind != LCC_ROUTER_SOFTMAX && l.e_router_kind != LCC_ROUTER_TOPK_SOFTMAX) return fail("unknown router kind");
             if (l.e_router_kind == LCC_ROUTER_TOPK_SOFTMAX && (l.e_identity > 0 || l.e_groups > 0 || l.e_shared_ff > 0))
                 return fail("routed feed-forward: weights over the chosen logits combine with neither identity experts, groups nor a shared expert");
-            if (l.e_act != LCC_EXPERT_RELU2 && l.e_act != LCC_EXPERT_CLAMP_GLU && l.e_act != LCC_EXPERT_SILU_GLU) return fail("unknown expert activation");
-            if (l.e_up_il16 && (l.e_act == LCC_EXPERT_RELU2 || l.e_ff % 16)) return fail("interleaved gate / up rows need a gated expert width that is a multiple of 16");
+            if (l.e_group_top < 0 || l.e_group_top > 2) return fail("routed feed-forward: a group scores as its best one or two scores");
+            if (l.e_act < LCC_EXPERT_RELU2 || l.e_act > LCC_EXPERT_GELU) return fail("unknown expert activation");
+            if (l.e_up_il16 && (l.e_act == LCC_EXPERT_RELU2 || l.e_act == LCC_EXPERT_GELU || l.e_ff % 16)) return fail("interleaved gate / up rows need a gated expert width that is a multiple of 16");
         } else if (l.ff_kind != LCC_FF_GLU && l.ff_kind != LCC_FF_MLP) {
             return fail("unknown feed-forward kind");
         }
         if (bn && l.canon_w_f32 && desc->canon_taps < 1) return fail("a convolution in front of the mixer needs its tap count");
         if (!l.norm1_f32 || (l.ff > 0 && ((!par && !l.norm2_f32) || !l.ff_in || !l.ff_out))) return fail("missing norm / feed-forward weights");
+        if (sw && (!l.norm1b_f32 || ((l.ff > 0 || l.ff_kind == LCC_FF_MOE) && !l.norm2b_f32))) return fail("missing norms behind the sublayers");
+        if (l.ff_kind == LCC_FF_MLP && l.ff_act != LCC_ACT_GELU_TANH && l.ff_act != LCC_ACT_RELU2) return fail("unknown feed-forward activation");
         if (dyt && !l.norm1_bias_f32) return fail("missing norm bias");
         if (par && l.type != LCC_MIX_ATTENTION) return fail("a parallel block takes the attention mixer");
-        if (!par && !bn && l.type == LCC_MIX_ATTENTION) return fail("the attention mixer is served in parallel blocks and in blocks normed on the sublayer's output");
-        if (bn && l.type == LCC_MIX_PARALLEL) return fail("the parallel mixer merges its branches in a post-norm block");
+        if (!par && !bn && !sw && l.type == LCC_MIX_ATTENTION) return fail("the attention mixer is not served in post-norm blocks and blocks on several streams");
+        if ((bn || sw) && l.type == LCC_MIX_PARALLEL) return fail("the parallel mixer merges its branches in a post-norm block");
         if (hc && (!l.hc1_f32 || ((l.ff > 0 || l.ff_kind == LCC_FF_MOE) && !l.hc2_f32))) return fail("missing stream weights");
         if (hc && l.type == LCC_MIX_PARALLEL) return fail("the parallel mixer merges its branches in a post-norm block");
         if (l.type == LCC_MIX_SSD) {
@@ -337,7 +347,10 @@ lcc_seq_model* lcc_seq_model_create(lcc_ctx* ctx, const lcc_seq_model_desc* desc
                 (l.m_rot_dims & 1) || l.m_rot_dims > l.m_dim || (l.m_value_keys && l.m_vdim != l.m_dim) || l.m_gate < LCC_GATE_NONE ||
                 l.m_gate > LCC_GATE_CHANNEL)
                 return fail("attention layer: unsupported sizes");
-            if (!l.m_in || (!l.m_unit_norm && (!l.m_qnorm_f32 || !l.m_knorm_f32)) || !l.m_out || (l.m_rot_dims > 0 && !l.rot_inv_freq_f32))
+            if (l.m_maps < 0 || l.m_maps > 2 || l.m_keep_first < 0 || (l.m_keep_first > 0 && l.m_chunk > 0) ||
+                (l.m_maps == 2 && (l.m_value_keys || l.m_gate != LCC_GATE_NONE || l.m_sink || l.m_rot_dims || !l.m_no_qk_norm || l.m_unit_norm || l.m_temp_f32)))
+                return fail("attention layer: unsupported options (two maps combine with projected values only: no norm, rotation, gate or sink)");
+            if (!l.m_in || (!l.m_unit_norm && !l.m_no_qk_norm && (!l.m_qnorm_f32 || !l.m_knorm_f32)) || !l.m_out || (l.m_rot_dims > 0 && !l.rot_inv_freq_f32))
                 return fail("attention layer: missing weights");
             if (l.m_vmix_role < 0 || l.m_vmix_role > 2 || (l.m_vmix_role && l.m_value_keys)) return fail("attention layer: values are mixed across layers only when they are projected");
             if (l.m_vmix_role == 1) {
@@ -439,17 +452,19 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
     uint8_t* o1 = ws + L.o1; uint8_t* o2 = ws + L.o2; uint8_t* xf = ws + L.xf;
     float* scan_ws = L.scan_floats ? (float*)(ws + L.scan) : nullptr;
     float* split_ws = L.split_floats ? (float*)(ws + L.split) : nullptr;
-    const bool hc = d.block == LCC_BLOCK_PRENORM_HC, par = d.block == LCC_BLOCK_PARALLEL, bn = d.block == LCC_BLOCK_BRANCHNORM;
+    const bool hc = d.block == LCC_BLOCK_PRENORM_HC, par = d.block == LCC_BLOCK_PARALLEL, bn = d.block == LCC_BLOCK_BRANCHNORM,
+               sw = d.block == LCC_BLOCK_SANDWICH;
     const int NS = hc ? d.streams : 1;
     uint8_t* vkeep = ws + L.vkeep;
     // blocks normed on the sublayer's output: does layer i read the residual stream through a convolution over time?
     auto canon_of = [&](int i) { return bn && i < d.n_layers && m->layers[i].canon_w_f32 != nullptr; };
-    // parallel blocks: the norm that opens layer i (none past the last layer)
+    // parallel and sandwich blocks: the norm that opens layer i (none past the last layer)
     auto norm_of = [&](int i) {
         if (i >= d.n_layers) return lcc::NormSpec{d.norm_kind, nullptr, nullptr, 0.f, d.eps};
         const lcc_seq_layer& n = m->layers[i];
         return lcc::NormSpec{d.norm_kind, n.norm1_f32, n.norm1_bias_f32, n.norm1_alpha, d.eps};
     };
+    auto spec_of = [&](const float* w) { return lcc::NormSpec{d.norm_kind, w, nullptr, 0.f, d.eps}; };
     float* xsum = (float*)(ws + L.xsum);
     // pre-norm blocks: the sublayer output that the next boundary kernel folds into the streams
     const float* pend_hc = nullptr;
@@ -479,7 +494,7 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
                                      pos_of(en), s, NS), "embedding");
             r0 += en.n_new;
         }
-        if (par) STEP(lcc::residual_norm(dt, x32, nullptr, 0, nullptr, 0, nullptr, norm_of(0), xa, T, W, s), "first norm");
+        if (par || sw) STEP(lcc::residual_norm(dt, x32, nullptr, 0, nullptr, 0, nullptr, norm_of(0), xa, T, W, s), "first norm");
     }
     for (int li = 0; li < d.n_layers; ++li) {
         const lcc_seq_layer& l = m->layers[li];
@@ -543,8 +558,9 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
                  "head norm + gate");
             STEP(linear(m, mid2, ldv, l.d_out, nullptr, o1, W, false, T, W, z.d_nv, s), "delta-rule out-proj");
         } else if (l.type == LCC_MIX_RETENTION) {
-            // [q | k | v | gate] -> rotary q, k (k scaled), everything that enters the recurrence packed as fp32 -> recurrence
-            // with one constant decay per head -> unit-rms heads x silu(gate) -> out-proj
+            // [q | k | v | gate] -> rotary q, k (k scaled) or silu on q, k, v, everything that enters the recurrence packed as fp32 ->
+            // recurrence with one constant decay per head -> unit-rms heads x silu(gate), or one norm over all heads with a weight x
+            // sigmoid(gate) -> out-proj
             const int ldp = ld8(z.t_proj), ldv = ld8(z.t_nv), H = l.t_heads;
             STEP(linear(m, xa, W, l.t_in, nullptr, proj, ldp, false, T, z.t_proj, W, s), "retention in-proj");
             int r0 = 0;
@@ -555,10 +571,11 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
                 st += st_off;
                 const lcc::SeqPos pos = pos_of(en);
                 float* pk = q32 + (size_t)r0 * z.t_pack;
+                const bool silu = l.t_silu != 0;
                 const lcc::RotarySegment seg[3] = {
-                    {0, 0, H, l.t_dim, 0, l.t_rot_dims, 1.f},
-                    {z.t_nk, z.t_nk, H, l.t_dim, 0, l.t_rot_dims, 1.f / sqrtf((float)l.t_dim)},
-                    {2 * z.t_nk, 2 * z.t_nk, H, l.t_vdim, 0, 0, 1.f}};
+                    {0, 0, H, l.t_dim, 0, l.t_rot_dims, 1.f, silu},
+                    {z.t_nk, z.t_nk, H, l.t_dim, 0, l.t_rot_dims, l.t_plain_keys ? 1.f : 1.f / sqrtf((float)l.t_dim), silu},
+                    {2 * z.t_nk, 2 * z.t_nk, H, l.t_vdim, 0, 0, 1.f, silu}};
                 STEP(lcc::rotary_pack_f32(dt, proj + (size_t)r0 * ldp * es, ldp, pk, z.t_pack, seg, 3, l.rot_inv_freq_f32, l.rot_mag,
                                           l.t_log_decay_f32, f1 + (size_t)r0 * H, H, en.n_new, pos, s), "rotary positions");
                 lcc::ScanArgs a{};
@@ -575,8 +592,9 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
                 STEP(lcc::gated_scan(a, pos, s), "retention recurrence");
                 r0 += en.n_new;
             }
-            STEP(lcc::gated_group_norm(dt, y32, z.t_nv, proj + (size_t)(2 * z.t_nk + z.t_nv) * es, ldp, l.t_norm_f32, l.t_vdim, mid2, ldv, T,
-                                       z.t_nv, l.t_vdim, 0, d.eps, s), "head norm + gate");
+            STEP(lcc::gated_group_norm(dt, y32, z.t_nv, proj + (size_t)(2 * z.t_nk + z.t_nv) * es, ldp, l.t_norm_f32,
+                                       l.t_whole_norm ? z.t_nv : l.t_vdim, mid2, ldv, T, z.t_nv, l.t_whole_norm ? z.t_nv : l.t_vdim,
+                                       l.t_gate_sigmoid ? 2 : 0, d.eps, s), "head norm + gate");
             STEP(linear(m, mid2, ldv, l.t_out, nullptr, o1, W, false, T, W, z.t_nv, s), "retention out-proj");
         } else if (l.type == LCC_MIX_LATENT) {
             // [q | latent, key part | gate] -> cache append + rotary query part -> unrotated query part absorbed through
@@ -594,7 +612,8 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
                 qsrc = proj2; ldq = ld8(z.a_nq);
             }
             const bool own_q = l.a_q_rank > 0;
-            const lcc::AttnOpts lo{l.a_window, l.a_sink_f32 == nullptr, false};
+            lcc::AttnOpts lo;
+            lo.window = l.a_window; lo.no_sink = l.a_sink_f32 == nullptr;
             int r0 = 0;
             for (int e = 0; e < n_entries; ++e) {
                 const lcc_seq_entry& en = entries[e];
@@ -622,8 +641,12 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
             // [q | k | (v) | gate] -> per-head q/k norm + rotary positions, k and the values (the key columns as projected, or
             // their own) into the pages -> attention inside the window -> sigmoid gate (in the attention kernel's store) -> out-proj
             const int ldp = ld8(z.m_proj), ldo = ld8(z.m_o);
-            STEP(linear(m, xa, W, l.m_in, nullptr, proj, ldp, false, T, z.m_proj, W, s), "attention in-proj");
-            const lcc::AttnOpts ao{l.m_window, !l.m_sink, l.m_gate == LCC_GATE_CHANNEL};
+            STEP(linear(m, xa, W, l.m_in, l.m_in_bias_f32, proj, ldp, false, T, z.m_proj, W, s, l.m_in_bias), "attention in-proj");
+            lcc::AttnOpts ao;
+            ao.window = l.m_window; ao.no_sink = !l.m_sink; ao.gate_channel = l.m_gate == LCC_GATE_CHANNEL;
+            ao.keep_first = l.m_keep_first; ao.softcap = l.m_softcap;
+            const int maps = l.m_maps > 1 ? l.m_maps : 1;
+            if (maps > 1) { ao.maps = maps; ao.lambda = l.m_lambda; ao.diff_scale = l.m_diff_scale; ao.eps = d.eps; }
             int r0 = 0;
             for (int e = 0; e < n_entries; ++e) {
                 const lcc_seq_entry& en = entries[e];
@@ -639,7 +662,8 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
                                           l.m_vmix_role == 1 ? vkeep + (size_t)r0 * ldk * es : nullptr, ldk};
                 STEP(lcc::qk_headnorm_rope_append(dt, pr, ldp, z.m_vcol, l.m_qnorm_f32, l.m_knorm_f32, d.eps, l.rot_inv_freq_f32, l.rot_mag,
                                                   l.m_rot_dims, l.m_rot_pairs, q, en.k_pages[li], en.v_pages[li], en.page_table, page_size,
-                                                  en.n_new, l.m_heads, l.m_kv_heads, l.m_dim, l.m_vdim, pos, s, &apo), "q/k norm + rotary + cache append");
+                                                  en.n_new, l.m_heads, l.m_kv_heads, maps * l.m_dim, l.m_vdim, pos, s, &apo), "q/k norm + rotary + cache append");
+                if (maps > 1) ao.raw = y32 + (size_t)r0 * l.m_heads * maps * l.m_vdim;
                 STEP(lcc::attn_masked(dt, q, en.k_pages[li], en.v_pages[li], en.page_table, page_size,
                                       z.m_ngate ? pr + (size_t)z.m_gate * es : nullptr, ldp, mid + (size_t)r0 * ldo * es, ldo, en.n_new,
                                       l.m_heads, l.m_kv_heads, l.m_dim, l.m_vdim, l.m_chunk, l.m_scale, m->use_tc, pos, s, ao, nullptr, 0,
@@ -741,10 +765,13 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
         else if (bn)       // x <- x + norm1(mixer); the feed-forward (or a next layer without a convolution) reads the new row
             STEP(lcc::branch_norm_residual(dt, x32, o1, W, nullptr, l.norm1_f32, d.eps, (has_ff || (li + 1 < d.n_layers && !canon_of(li + 1))) ? xa : nullptr,
                                            T, W, s), "norm1 + residual");
+        else if (sw)       // x <- x + norm1b(mixer), then the norm that the feed-forward (or the next layer) reads
+            STEP(lcc::sandwich_residual(dt, x32, o1, W, nullptr, spec_of(l.norm1b_f32), has_ff ? spec_of(l.norm2_f32) : norm_of(li + 1), xa, T, W, s),
+                 "norm1b + residual + next norm");
         else if (l.type != LCC_MIX_PARALLEL)
             STEP(lcc::postnorm_residual(dt, x32, xa, o1, W, nullptr, nullptr, 0, nullptr, l.norm1_f32, d.alpha, d.eps, T, W, s), "norm1");
         if (has_ff && hc) STEP(boundary(l.hc2_f32, l.norm2_f32, nullptr), "stream boundary");
-        lcc::MoeCombine par_mc{};       // parallel block and output-normed block: the routed feed-forward's row is formed by the layer's residual kernel
+        lcc::MoeCombine par_mc{};       // parallel, output-normed and sandwich blocks: the routed feed-forward's row is formed by the layer's residual kernel
         bool par_is_mc = false;
         if (l.ff_kind == LCC_FF_MOE) {
             // E real experts own row lists; the router has EO = E + identity outputs
@@ -754,8 +781,9 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
             const float glu_limit = silu_glu ? INFINITY : l.e_limit, glu_alpha = silu_glu ? 1.f : 1.702f, glu_up_bias = silu_glu ? 0.f : 1.f;
             const int E = l.e_experts, EO = E + l.e_identity, K = l.e_top, lde = ld8(EO + 1), NH = glu ? 2 * l.e_ff : l.e_ff, ldh = ld8(NH),
                       ldg = ld8(l.e_ff), ldw8 = ld8(W), lds = ld8(l.e_shared_ff);
-            const lcc::MoeRouterOpts ro{l.e_router_kind == LCC_ROUTER_SOFTMAX, l.e_identity, l.e_groups, l.e_keep, l.e_router_kind == LCC_ROUTER_TOPK_SOFTMAX};
-            const int up_act = glu ? lcc::ACT_NONE : lcc::ACT_RELU2;
+            const lcc::MoeRouterOpts ro{l.e_router_kind == LCC_ROUTER_SOFTMAX, l.e_identity, l.e_groups, l.e_keep, l.e_router_kind == LCC_ROUTER_TOPK_SOFTMAX,
+                                       l.e_group_top > 1 ? l.e_group_top : 1};
+            const int up_act = glu ? lcc::ACT_NONE : (l.e_act == LCC_EXPERT_GELU ? lcc::ACT_GELU_ERF : lcc::ACT_RELU2);
             float* mf = (float*)(ws + L.moe_f);
             float* logit = mf; float* wsel = mf + (size_t)T * lde; float* sgate = wsel + (size_t)T * K;
             int* mi = (int*)(ws + L.moe_i);
@@ -763,7 +791,8 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
             int* tile_group = src_row + L.moe_rows; int* counts = tile_group + L.moe_rows / kMoeTile + 1; int* row_off = counts + E;
             uint8_t* ex = ws + L.moe_x; uint8_t* eh = ws + L.moe_h; uint8_t* eg = ws + L.moe_g; uint8_t* eo = ws + L.moe_o;
             const bool shared = l.e_shared_ff > 0, ident = l.e_identity > 0;
-            float* gate_out = (shared || ident) ? sgate : nullptr;   // the shared expert's gate, or the chosen identity experts' weights
+            const bool sh_gate = shared && !l.e_shared_ungated;
+            float* gate_out = (sh_gate || ident) ? sgate : nullptr;   // the shared expert's gate, or the chosen identity experts' weights
             // experts on the tensor cores: bf16, enough routed rows, 8-aligned shapes; lists are then padded to whole tiles
             const bool tc = m->use_tc && dt == LCC_DT_BF16 && T * K >= kMoeTcMinRows && (W % 8) == 0 && (l.e_ff % 8) == 0 && W >= 64 && l.e_ff >= 64;
             const int rows_max = T * K + E * (kMoeTile - 1), n_tiles = (rows_max + kMoeTile - 1) / kMoeTile;
@@ -774,11 +803,12 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
                 LCC_FAIL(m->ctx, -100, "stream fork failed");
             if (shared) {
                 cudaStream_t ss = fork ? m->side : fs;
-                STEP(linear(m, xa, W, l.e_shared_up, nullptr, mid2, lds, false, T, l.e_shared_ff, W, ss, nullptr, lcc::ACT_RELU2), "shared expert up");
+                STEP(linear(m, xa, W, l.e_shared_up, nullptr, mid2, lds, false, T, l.e_shared_ff, W, ss, nullptr,
+                            l.e_act == LCC_EXPERT_GELU ? lcc::ACT_GELU_ERF : lcc::ACT_RELU2), "shared expert up");
                 STEP(linear(m, mid2, lds, l.e_shared_down, nullptr, o2, W, false, T, W, l.e_shared_ff, ss), "shared expert down");
             }
             // router logits (and the shared expert's gate logit) accumulate in fp32 from the normed row
-            STEP(linear(m, xa, W, l.e_router, nullptr, logit, lde, true, T, EO + (shared ? 1 : 0), W, fs), "router");
+            STEP(linear(m, xa, W, l.e_router, nullptr, logit, lde, true, T, EO + (sh_gate ? 1 : 0), W, fs), "router");
             if (!tc && T * K <= 256 && EO <= 512) {
                 STEP(lcc::moe_route_small(logit, lde, l.e_correction_f32, EO, K, l.e_scale, sel, wsel, gate_out, row_off, posn,
                                           src_row, T, fs, &ro), "expert choice + row lists");
@@ -796,7 +826,7 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
                 a.A = ex; a.B = l.e_up; a.C = epi_glu ? eg : eh; a.M = n_tiles * kMoeTile; a.N = NH; a.K = W; a.lda = ldw8; a.ldb = W;
                 a.ldc = epi_glu ? ldg : ldh;
                 a.bias = nullptr; a.residual = nullptr; a.ldr = 0; a.block_n = 0;
-                a.epi = epi_glu ? lcc::EPI_CLAMP_GLU : (glu ? lcc::EPI_NONE : lcc::EPI_RELU2);
+                a.epi = epi_glu ? lcc::EPI_CLAMP_GLU : (glu ? lcc::EPI_NONE : (l.e_act == LCC_EXPERT_GELU ? lcc::EPI_GELU_ERF : lcc::EPI_RELU2));
                 a.epi_param = glu_limit; a.epi_alpha = glu_alpha; a.epi_up_bias = glu_up_bias;
                 a.tile_group = tile_group; a.groups = E;
                 STEP(lcc::gemm_bf16_tn(a, m->ctx->num_sms, fs), "experts up");
@@ -823,18 +853,19 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
             if (fork && (cudaEventRecord(m->ev_join, m->side) != cudaSuccess || cudaStreamWaitEvent(fs, m->ev_join, 0) != cudaSuccess))
                 LCC_FAIL(m->ctx, -100, "stream join failed");
             if (hc) {   // the weighted sum of the experts' rows is formed by the boundary kernel that folds it into the streams
-                pend_mc = lcc::MoeCombine{eo, ldw8, posn, wsel, K, shared ? o2 : nullptr, W, sgate};
+                pend_mc = lcc::MoeCombine{eo, ldw8, posn, wsel, K, shared ? o2 : nullptr, W, gate_out};
                 pend_is_mc = true;
-            } else if (par || bn) {   // ... or by the residual kernel that closes the layer; identity experts return the normed row
-                par_mc = lcc::MoeCombine{eo, ldw8, posn, wsel, K, shared ? (const void*)o2 : (ident ? (const void*)xa : nullptr), W, sgate};
+            } else if (par || bn || sw) {   // ... or by the residual kernel that closes the layer; identity experts return the normed row
+                par_mc = lcc::MoeCombine{eo, ldw8, posn, wsel, K, shared ? (const void*)o2 : (ident ? (const void*)xa : nullptr), W, gate_out};
                 par_is_mc = true;
             } else {
-                STEP(lcc::moe_combine(dt, eo, ldw8, posn, wsel, K, shared ? o2 : nullptr, W, sgate, o1, W, T, W, fs), "expert combine");
+                STEP(lcc::moe_combine(dt, eo, ldw8, posn, wsel, K, shared ? o2 : nullptr, W, gate_out, o1, W, T, W, fs), "expert combine");
             }
         } else if (l.ff > 0 && l.ff_kind == LCC_FF_MLP) {
             const int ldf = ld8(l.ff);
             // (its hidden rows in mid2: in a parallel block the mixer's rows in mid may still be in use on the other stream)
-            STEP(linear(m, xa, W, l.ff_in, nullptr, mid2, ldf, false, T, l.ff, W, fs, nullptr, lcc::ACT_GELU_TANH), "feed-forward up + gelu");
+            STEP(linear(m, xa, W, l.ff_in, nullptr, mid2, ldf, false, T, l.ff, W, fs, nullptr,
+                        l.ff_act == LCC_ACT_RELU2 ? lcc::ACT_RELU2 : lcc::ACT_GELU_TANH), "feed-forward up + activation");
             STEP(linear(m, mid2, ldf, l.ff_out, nullptr, par ? o2 : o1, W, false, T, W, l.ff, fs), "feed-forward down");
         } else if (l.ff > 0) {
             const int ldg = ld8(2 * l.ff), ldf = ld8(l.ff);
@@ -852,6 +883,10 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
             // x <- x + norm2(feed-forward); a next layer without a convolution in front of its mixer reads the new row
             STEP(lcc::branch_norm_residual(dt, x32, par_is_mc ? nullptr : o1, W, par_is_mc ? &par_mc : nullptr, l.norm2_f32, d.eps,
                                            (li + 1 < d.n_layers && !canon_of(li + 1)) ? xa : nullptr, T, W, s), "norm2 + residual");
+        } else if (has_ff && sw) {
+            // x <- x + norm2b(feed-forward), then the next layer's first norm of the new row
+            STEP(lcc::sandwich_residual(dt, x32, par_is_mc ? nullptr : o1, W, par_is_mc ? &par_mc : nullptr, spec_of(l.norm2b_f32), norm_of(li + 1),
+                                        xa, T, W, s), "norm2b + residual + next norm");
         } else if (has_ff) {
             if (hc) pend_hc = l.hc2_f32;
             else STEP(lcc::postnorm_residual(dt, x32, xa, o1, W, nullptr, nullptr, 0, nullptr, l.norm2_f32, d.alpha, d.eps, T, W, s), "norm2");

@@ -29,7 +29,7 @@ struct SeqPos {
 };
 
 // The row a routed feed-forward contributes, formed inside the kernel that consumes it (hyper_boundary, residual_norm):
-//   y[r] = sum_k weight[r, k] * eo[pos[r, k]] + gate[r] * so[r]   (fp32; choices with pos < 0 are skipped)
+//   y[r] = sum_k weight[r, k] * eo[pos[r, k]] + gate[r] * so[r]   (fp32; choices with pos < 0 are skipped; gate null: 1)
 struct MoeCombine {
     const void* eo; int ld_eo; const int* pos; const float* weight; int top;
     const void* so; int ld_so; const float* gate;      // so null: no shared expert
@@ -64,7 +64,7 @@ struct GroupedLinear {
     // the defaults are the clamped form above; alpha 1, up_bias 0 and an infinite limit give silu(gate) * up
     float glu_alpha = 1.702f, glu_up_bias = 1.f;
 };
-enum { ACT_NONE = 0, ACT_RELU2 = 1, ACT_GELU_TANH = 2 };   // 2: 0.5 x (1 + tanh(sqrt(2/pi) (x + 0.044715 x^3)))
+enum { ACT_NONE = 0, ACT_RELU2 = 1, ACT_GELU_TANH = 2, ACT_GELU_ERF = 3 };   // 3: 0.5 x (1 + erf(x / sqrt(2))); 2: 0.5 x (1 + tanh(sqrt(2/pi) (x + 0.044715 x^3)))
 int linear_grouped(const GroupedLinear& g, cudaStream_t s);
 
 // ---- recurrent.cu -------------------------------------------------------------------------------------------------------
@@ -193,8 +193,20 @@ int attn_chunk_sink(int dt, const float* q, const void* k_pages, const void* v_p
 size_t attn_split_ws_floats(int rows, int Hq, int DV);
 // Further options of attn_chunk_sink (null: chunks only, a zero-logit sink, one gate per head). window > 0: a row at position
 // i sees only j with i - j < window (inside its chunk, when there are chunks too). no_sink: ordinary softmax over the visible
-// keys. gate_channel: the gate slice is [S, Hq*DV], one sigmoid gate per output element.
-struct AttnOpts { int window; bool no_sink; bool gate_channel; };
+// keys. gate_channel: the gate slice is [S, Hq*DV], one sigmoid gate per output element. keep_first: positions j < keep_first stay
+// visible behind the window. softcap > 0: a score s becomes softcap * tanh(s / softcap). maps = 2 (differential attention; no gate):
+// q is [S, Hq, 2, D] and a K row holds the two maps of a key/value head (2 * D channels); each map is a softmax of its own over the
+// same values, and the head's output is rms(a1 - lambda * a2) * diff_scale over its DV channels (x / sqrt(mean(x^2) + eps)). raw: fp32
+// [S, Hq, 2, DV] scratch for the kernels that do not form the difference themselves (given with maps = 2 only).
+struct AttnOpts {
+    int window = 0;
+    bool no_sink = false, gate_channel = false;
+    int keep_first = 0;
+    float softcap = 0.f;
+    int maps = 1;
+    float lambda = 0.f, diff_scale = 1.f, eps = 0.f;
+    float* raw = nullptr;
+};
 // Options of qk_headnorm_rope_append (null: none). unit_norm: q and k heads are divided by their rms without a weight (qn_w, kn_w
 // null; the rotation keeps every pair's length, so norming before it equals norming after it). q_head_scale: fp32 [Hq], one factor
 // per query head on q_out (a temperature on the scores). v_mix: [S, ld_mix] slice (storage dt) of G*DV columns: the cached values
@@ -219,8 +231,9 @@ int qk_headnorm_rope_append(int dt, const void* proj, int ld, int v_col, const f
 // i + dims/2; the pair (u, v) at position p becomes (u cos a - v sin a, v cos a + u sin a) * mag, a = p * inv_freq[i]
 // (fp32 position, angle, cos and sin). A segment is `heads` heads of `dim` channels starting at column `col_in` of a row
 // of `in` (storage dt); the rotated block is channels [rot_off, rot_off + rot_dims) of each head, the rest pass; every
-// output is multiplied by `scale` and written as fp32 at column col_out of `out` with the same head layout.
-struct RotarySegment { int col_in, col_out, heads, dim, rot_off, rot_dims; float scale; };
+// output is multiplied by `scale` and written as fp32 at column col_out of `out` with the same head layout. silu: x * sigmoid(x) on
+// every input first.
+struct RotarySegment { int col_in, col_out, heads, dim, rot_off, rot_dims; float scale; bool silu = false; };
 // Up to 4 segments of one row in one launch. fill: optional fp32 [fill_n] row that is copied to fill_out [S, fill_n] for
 // every row (per-head constants a recurrence wants per token, e.g. log decays).
 int rotary_pack_f32(int dt, const void* in, int ld_in, float* out, int ld_out, const RotarySegment* seg, int n_seg,
@@ -261,8 +274,9 @@ int hyper_boundary(int dt, float* xs, int n, const void* y, int ld_y, const floa
 // must then be given; the logits have no shared-gate column); groups > 0: the E outputs form that many equal groups of
 // neighbours, a group scores as its largest choice score and only members of the `keep` best groups can be chosen.
 // topk_softmax: the choice is by logit (+ correction) and the weights are the softmax over the chosen logits only (times scale);
-// it combines with neither identity experts nor groups. correction may be null (zeros).
-struct MoeRouterOpts { bool softmax; int identity; int groups; int keep; bool topk_softmax = false; };
+// it combines with neither identity experts nor groups. correction may be null (zeros). group_top: a group scores as the sum of that
+// many of its largest choice scores (1 or 2).
+struct MoeRouterOpts { bool softmax; int identity; int groups; int keep; bool topk_softmax = false; int group_top = 1; };
 int moe_route(const float* logits, int ld, const float* correction, int E, int top, float scale, int* sel, float* weight,
               float* shared_gate, int* counts, int* rank, int S, cudaStream_t s, const MoeRouterOpts* opt = nullptr);
 // moe_route and moe_index (dense lists) in one launch of one CTA, for calls of up to kMoeSmallItems (row, choice) pairs; it
@@ -295,7 +309,7 @@ int postnorm_residual(int dt, float* x32, void* xa, const void* a, int ld_a, con
                       const float* wb, const float* w, float alpha, float eps, int S, int W, cudaStream_t s);
 // Grouped RMS norm with a multiplicative silu gate: y: fp32 [S, n]; gate: [S, n] slice (storage dt). Groups of `group`
 // consecutive columns; weight w[c % w_len]. gate_first 1: out = rms(y * silu(g)) * w; 0: out = rms(y) * w * silu(g);
-// 2: out = rms(y) * w * sigmoid(g).
+// 2: out = rms(y) * w * sigmoid(g). group = n: one norm over the whole row.
 int gated_group_norm(int dt, const float* y, int ld_y, const void* gate, int ld_gate, const float* w, int w_len,
                      void* out, int ld_out, int S, int n, int group, int gate_first, float eps, cudaStream_t s);
 // out[r, c] = gelu_tanh(gu[r, c]) * gu[r, F + c]
@@ -306,7 +320,8 @@ int gather_rmsnorm(int dt, const float* x32, const int* rows, const float* w, fl
 // out[r, :n] = rms(in[r, :n]) * w for a slice of rows in the storage type (in, out: leading dimensions in elements; w: fp32 [n])
 int slice_rmsnorm(int dt, const void* in, int ld_in, const float* w, float eps, void* out, int ld_out, int S, int n, cudaStream_t s);
 // A row norm: NORM_RMS x / sqrt(mean(x^2) + eps) * w; NORM_DYT tanh(alpha * x) * w + b (no statistics of the row).
-enum { NORM_RMS = 0, NORM_DYT = 1 };
+// NORM_LAYER (x - mean) / sqrt(mean squared deviation + eps) * w.
+enum { NORM_RMS = 0, NORM_DYT = 1, NORM_LAYER = 2 };
 struct NormSpec { int kind; const float* w; const float* b; float alpha; float eps; };
 // out[i, :] = norm(x32[rows[i], :])  (storage dt)
 int gather_norm(int dt, const float* x32, const int* rows, const NormSpec& n, void* out, int n_rows, int W, cudaStream_t s);
@@ -325,6 +340,10 @@ int glu_clamp_swish(int dt, const void* gu, int ld, void* out, int ld_out, int S
 // storage dt, what the next sublayer reads.
 int branch_norm_residual(int dt, float* x32, const void* a, int ld_a, const MoeCombine* mc, const float* w, float eps, void* xa,
                          int S, int W, cudaStream_t s);
+// A sublayer with a norm on either side, fused with the next sublayer's first norm: x32 <- x32 + post(y) in fp32, y as in
+// branch_norm_residual; then, if next.w, xa = next(x32) (storage dt). post and next: NORM_RMS or NORM_LAYER.
+int sandwich_residual(int dt, float* x32, const void* a, int ld_a, const MoeCombine* mc, const NormSpec& post, const NormSpec& next, void* xa,
+                      int S, int W, cudaStream_t s);
 // x <- cap * tanh(x / cap) in place (fp32; cap <= 0: unchanged), then x <- x * scale
 int softcap(float* x, int64_t n, float cap, cudaStream_t s, float scale = 1.f);
 

@@ -197,8 +197,9 @@ class SeqStatePool(PageAllocator):
       reads another layer's cache has no entry here.
     * Recurrent layers: one fp32 slot per sequence and layer (`state_floats[i]` elements, 0 for none), zeroed when a
       sequence takes it.
-    attn_layers: {layer index: (kv_heads, dim, vdim, chunk[, window])}; state_floats: per layer. A layer with a sliding
-    window of w positions never looks more than w - 1 positions behind the newest token."""
+    attn_layers: {layer index: (kv_heads, dim, vdim, chunk[, window[, keep_first]])}; state_floats: per layer. A layer with a
+    sliding window of w positions never looks more than w - 1 positions behind the newest token, but for the first `keep_first`
+    positions of the sequence, which stay: the pages between the two go back."""
 
     def __init__(self, attn_layers: dict, state_floats: List[int], dtype, device, initial_pages: int = 32, initial_slots: int = 2):
         self.attn_layers = dict(attn_layers)
@@ -229,12 +230,16 @@ class SeqStatePool(PageAllocator):
         if not self.attn_layers:
             return seq_len
         lo = seq_len
-        for (_g, _d, _dv, chunk, *rest) in self.attn_layers.values():
+        for (_g, _d, _dv, chunk, *rest) in self.attn_layers.values():     # (positions kept at the front: kept_first)
             first = (seq_len // chunk) * chunk if chunk > 0 else 0
             if rest and rest[0] > 0:       # the next token sits at position seq_len and sees seq_len - window + 1 onwards
                 first = max(first, seq_len - rest[0] + 1)
             lo = min(lo, first)
         return lo
+
+    def kept_first(self) -> int:
+        """Positions at the front of a sequence that some windowed layer reads for good."""
+        return max([rest[1] for (_g, _d, _dv, _c, *rest) in self.attn_layers.values() if len(rest) > 1 and rest[0] > 0] or [0])
 
     # state slots ------------------------------------------------------------------------------
     def _grow_slots(self, new_total: int):
@@ -314,11 +319,12 @@ class SeqCache:
     def advance(self, n_new: int):
         """`n_new` more tokens are cached; pages every attention layer has left go back to the pool."""
         self.seq_len += n_new
+        first_dead = (self.pool.kept_first() + PAGE_SIZE - 1) // PAGE_SIZE
         last_dead = self.pool.keep_from(self.seq_len) // PAGE_SIZE
-        dead = [p for p in self.pages[:last_dead] if p is not None]
+        dead = [p for p in self.pages[first_dead:last_dead] if p is not None]
         if dead:
             self.pool.release(dead)
-            for i in range(min(last_dead, len(self.pages))):
+            for i in range(first_dead, min(last_dead, len(self.pages))):
                 self.pages[i] = None
 
     def live_pages(self) -> int:

@@ -25,6 +25,7 @@ register("Bimopel", "livecc_b200.seq_engine", "SeqLMForCausalLM")
 register("Kedelorn", "livecc_b200.seq_engine", "SeqLMForCausalLM")
 register("Dibedra", "livecc_b200.seq_engine", "SeqLMForCausalLM")
 register("Lugizen", "livecc_b200.seq_engine", "SeqLMForCausalLM")
+register("Kapitar", "livecc_b200.seq_engine", "SeqLMForCausalLM")
 
 
 def architectures() -> list:

@@ -1,7 +1,7 @@
 """Hybrid sequence models (decoder-only language models built from state-space, gated-linear-attention, delta-rule, chunk-local
-attention, retention, latent-attention and sliding-window attention mixers, in post-norm blocks, pre-norm blocks on several
-residual streams, parallel blocks or blocks normed on the sublayer's output, with dense or routed feed-forwards) behind the same surface as the video-language engine: `from_pretrained`, `generate`, a cache object that
-callers pass back, greedy token selection in the library's sampling kernel.
+attention, retention, lightning, latent-attention, sliding-window and differential attention mixers, in post-norm blocks, pre-norm
+blocks on several residual streams, parallel blocks, blocks normed on the sublayer's output or on either side of it, with dense or
+routed feed-forwards) behind the same surface as the video-language engine: `from_pretrained`, `generate`, a cache object that callers pass back, greedy token selection in the library's sampling kernel.
 
     model = SeqLMForCausalLM.from_pretrained(path, torch_dtype="bfloat16", device_map="cuda")
     out = model.generate(input_ids, max_new_tokens=16)            # out.sequences, out.past_key_values
@@ -101,10 +101,10 @@ class SeqWeights:
 
         W = cfg.width
         self.embed = mat("embed")
-        self.head = mat("head")
+        self.head = self.embed if cfg.tied_head else mat("head")
         self.final_norm = norm_w("final.norm")
         self.final_norm_bias, self.final_norm_alpha = norm_extra("final.norm")
-        if shape("embed") != (cfg.vocab, W) or shape("head") != (cfg.vocab, W):
+        if shape("embed") != (cfg.vocab, W) or (not cfg.tied_head and shape("head") != (cfg.vocab, W)):
             raise ValueError("embed / head do not have the shape [vocab, width] of config.json")
         self.inv_freq = None
         if cfg.positions == "sinusoid":
@@ -119,6 +119,10 @@ class SeqWeights:
             p = f"l{i}."
             w = {"norm1": norm_w(p + "norm1")}
             w["norm1_bias"], w["norm1_alpha"] = norm_extra(p + "norm1")
+            if cfg.block == "sandwich":
+                w["norm1b"] = norm_w(p + "norm1b")
+                if L.ff or L.moe:
+                    w["norm2b"] = norm_w(p + "norm2b")
             if hc:
                 n = cfg.streams
                 for q in ("hc1", "hc2") if (L.ff or L.moe) else ("hc1",):
@@ -144,14 +148,18 @@ class SeqWeights:
                 w["d_conv_w"] = f32(segments([m + "q.conv", m + "k.conv", m + "v.conv"]))
                 w["d_a_up"], w["d_g_up"], w["d_out"] = mat(m + "a2"), mat(m + "g2"), mat(m + "o")
                 w["d_dt_bias"], w["d_a_log"], w["d_norm"] = f32(get(m + "dt_bias")), f32(get(m + "A_log")), f32(get(m + "norm"))
-            elif L.type == "retention":
+            elif L.type in ("retention", "lightning"):
                 rt, m = L.retention, p + "mix."
                 check(m + "q", (rt.heads * rt.dim, W)), check(m + "k", (rt.heads * rt.dim, W))
                 check(m + "v", (rt.heads * rt.vdim, W)), check(m + "g", (rt.heads * rt.vdim, W)), check(m + "o", (W, rt.heads * rt.vdim))
                 w["t_in"] = mat(m + "q", m + "k", m + "v", m + "g")
                 w["t_out"] = mat(m + "o")
                 w["t_log_decay"] = torch.log(torch.tensor(rt.decay, dtype=torch.float64)).to(torch.float32).to(device)
-                w["t_norm"] = torch.ones(rt.vdim, dtype=torch.float32, device=device)
+                if rt.whole_norm:
+                    check(m + "norm", (rt.heads * rt.vdim,))
+                    w["t_norm"] = f32(get(m + "norm"))
+                else:
+                    w["t_norm"] = torch.ones(rt.vdim, dtype=torch.float32, device=device)
                 if rt.rot.dims:
                     w["rot_freq"], w["rot_mag"] = rotary(rt.rot)
             elif L.type == "latent_attention":
@@ -185,8 +193,13 @@ class SeqWeights:
                 w["rot_freq"], w["rot_mag"] = rotary(a.rot)
             elif L.type == "attention":
                 a, m = L.attn, p + "mix."
-                check(m + "q", (a.heads * a.dim, W)), check(m + "k", (a.kv_heads * a.dim, W)), check(m + "o", (W, a.heads * a.vdim))
-                if not a.unit_norm:
+                check(m + "q", (a.heads * a.maps * a.dim, W)), check(m + "k", (a.kv_heads * a.maps * a.dim, W)), check(m + "o", (W, a.heads * a.vdim))
+                if a.maps > 1:      # the second map's weight: one number for the layer
+                    dot = lambda u, v: (get(m + u).to(torch.float64) * get(m + v).to(torch.float64)).sum()
+                    for n in ("lq1", "lk1", "lq2", "lk2"):
+                        check(m + n, (a.dim,))
+                    w["m_lambda"] = float(torch.exp(dot("lq1", "lk1")) - torch.exp(dot("lq2", "lk2"))) + a.diff
+                if a.qk_norm and not a.unit_norm:
                     check(m + "q.norm", (a.dim,)), check(m + "k.norm", (a.dim,))
                     w["m_qnorm"], w["m_knorm"] = f32(get(m + "q.norm")), f32(get(m + "k.norm"))
                 if a.temp:
@@ -206,6 +219,13 @@ class SeqWeights:
                     check(m + "g", (a.gate_rows, W))
                     rows.append(m + "g")
                 w["m_in"] = mat(*rows)
+                if a.bias:
+                    blocks = [get(n + ".b").float().reshape(-1) for n in rows[: 2 if a.value_keys else 3]]
+                    for n, b in zip(rows, blocks):
+                        check(n + ".b", (shape(n)[0],))
+                    bias = torch.cat(blocks)
+                    bias = torch.cat([bias, torch.zeros(w["m_in"].shape[0] - bias.numel(), device=bias.device)])
+                    w["m_in_bias"], w["m_in_bias_st"] = f32(bias), bias.to(device=device, dtype=dtype).contiguous()
                 w["m_out"] = mat(m + "o")
                 if a.rot.dims:
                     w["rot_freq"], w["rot_mag"] = rotary(a.rot)
@@ -259,7 +279,7 @@ class SeqWeights:
                 for j in range(e.experts):
                     check(f"{m}e{j}.up", (e.ff, W)), check(f"{m}e{j}.down", (W, e.ff))
                 check(m + "router", (e.outputs, W))
-                if e.router != "topk_softmax":
+                if e.router != "topk_softmax" and e.correction:
                     check(m + "correction", (e.outputs,))
                 if e.act in ("clamp_glu", "silu_glu"):
                     # each expert's gate and up rows in one matrix, so that one product per expert list yields both. Widths that
@@ -279,11 +299,13 @@ class SeqWeights:
                 else:
                     w["e_up"] = torch.stack([get(f"{m}e{j}.up") for j in range(e.experts)]).to(device=device, dtype=dtype).contiguous()
                 w["e_down"] = torch.stack([get(f"{m}e{j}.down") for j in range(e.experts)]).to(device=device, dtype=dtype).contiguous()
-                if e.router != "topk_softmax":
+                if e.router != "topk_softmax" and e.correction:
                     w["e_correction"] = f32(get(m + "correction"))
                 if e.shared_ff:
-                    check(m + "shared.up", (e.shared_ff, W)), check(m + "shared.down", (W, e.shared_ff)), check(m + "shared.sg", (1, W))
-                    w["e_router"] = mat(m + "router", m + "shared.sg")     # the shared gate's logit is one more router row
+                    check(m + "shared.up", (e.shared_ff, W)), check(m + "shared.down", (W, e.shared_ff))
+                    if e.shared_gate:
+                        check(m + "shared.sg", (1, W))
+                    w["e_router"] = mat(m + "router", m + "shared.sg") if e.shared_gate else mat(m + "router")   # the shared gate's logit is one more router row
                     w["e_shared_up"], w["e_shared_down"] = mat(m + "shared.up"), mat(m + "shared.down")
                 else:
                     w["e_router"] = mat(m + "router")
@@ -304,7 +326,7 @@ class SeqWeights:
         self.unused = sorted(set(t) - used)
 
     def nbytes(self) -> int:
-        n = sum(x.numel() * x.element_size() for x in (self.embed, self.head, self.final_norm))
+        n = sum(x.numel() * x.element_size() for x in {id(x): x for x in (self.embed, self.head, self.final_norm)}.values())
         own = {id(w): w for w in self.layers}.values()      # layers that share tensors count once
         return n + sum(x.numel() * x.element_size() for w in own for x in w.values() if isinstance(x, torch.Tensor))
 
@@ -321,8 +343,8 @@ class SeqLMForCausalLM:
         self.ctx = _cabi.Context(device.index if device.index is not None else torch.cuda.current_device(), profile=self.PROFILE)
         self._native = self._build_native()
         attn = {i: (L.left.kv_heads, L.left.dim, L.left.vdim, L.left.chunk) for i, L in enumerate(config.layers) if L.type == "parallel"}
-        # sliding-window attention: (kv heads, key size, value size, no chunks, window)
-        attn.update({i: (L.attn.kv_heads, L.attn.dim, L.attn.vdim, 0, L.attn.window) for i, L in enumerate(config.layers) if L.type == "attention"})
+        # sliding-window attention: (kv heads, key size (both maps of a differential head), value size, no chunks, window, kept first positions)
+        attn.update({i: (L.attn.kv_heads, L.attn.maps * L.attn.dim, L.attn.vdim, 0, L.attn.window, L.attn.keep_first) for i, L in enumerate(config.layers) if L.type == "attention"})
         # a latent cache is one K pool of [latent | rotary key part] rows; a layer that reads another layer's cache has none
         attn.update({i: (1, L.latent.kv_rank + L.latent.rot_dim, 0, 0, L.latent.window) for i, L in enumerate(config.layers)
                      if L.type == "latent_attention" and L.latent.kv_from < 0})
@@ -346,7 +368,7 @@ class SeqLMForCausalLM:
     @classmethod
     def from_pretrained(cls, model_path: str, torch_dtype="auto", device_map="cuda", max_tokens: int = 0, **_):
         """A directory with config.json and *.safetensors (bf16 tensors; names `embed`, `l<i>.norm1`, `l<i>.mix.*`,
-        `l<i>.mlp.*`, `final.norm`, `head`; a Dynamic-Tanh norm adds `<norm>.b` and `<norm>.alpha`)."""
+        `l<i>.mlp.*`, `final.norm`, `head` unless the embedding table is the head; a Dynamic-Tanh norm adds `<norm>.b` and `<norm>.alpha`)."""
         from .checkpoint import iter_safetensors
 
         with open(os.path.join(model_path, "config.json")) as f:
@@ -363,6 +385,7 @@ class SeqLMForCausalLM:
             e.ff = L.ff
             e.norm1_f32 = p(lw["norm1"])
             e.norm1_bias_f32, e.norm1_alpha = p(lw.get("norm1_bias")), lw.get("norm1_alpha", 0.0)
+            e.norm1b_f32, e.norm2b_f32 = p(lw.get("norm1b")), p(lw.get("norm2b"))
             e.hc1_f32, e.hc2_f32 = p(lw.get("hc1")), p(lw.get("hc2"))
             e.a_kv_from = -1
             e.rot_inv_freq_f32, e.rot_mag = p(lw.get("rot_freq")), lw.get("rot_mag", 1.0)
@@ -373,9 +396,10 @@ class SeqLMForCausalLM:
                 e.d_heads, e.d_kv_heads, e.d_dim, e.d_vdim, e.d_conv, e.d_rank_a, e.d_rank_g = t.heads, t.kv_heads, t.dim, t.vdim, t.conv, t.rank_a, t.rank_g
                 e.d_in, e.d_conv_w_f32, e.d_a_up, e.d_g_up, e.d_out = p(lw["d_in"]), p(lw["d_conv_w"]), p(lw["d_a_up"]), p(lw["d_g_up"]), p(lw["d_out"])
                 e.d_dt_bias_f32, e.d_a_log_f32, e.d_norm_f32 = p(lw["d_dt_bias"]), p(lw["d_a_log"]), p(lw["d_norm"])
-            elif L.type == "retention":
+            elif L.type in ("retention", "lightning"):
                 t = L.retention
                 e.type = _cabi.MIX_RETENTION
+                e.t_silu, e.t_plain_keys, e.t_whole_norm, e.t_gate_sigmoid = int(t.silu), int(not t.key_scale), int(t.whole_norm), int(t.gate == "sigmoid")
                 e.t_heads, e.t_dim, e.t_vdim, e.t_rot_dims = t.heads, t.dim, t.vdim, t.rot.dims
                 e.t_in, e.t_log_decay_f32, e.t_norm_f32, e.t_out = p(lw["t_in"]), p(lw["t_log_decay"]), p(lw["t_norm"]), p(lw["t_out"])
             elif L.type == "latent_attention":
@@ -395,6 +419,9 @@ class SeqLMForCausalLM:
                 e.m_gate = {"none": _cabi.GATE_NONE, "head": _cabi.GATE_HEAD, "channel": _cabi.GATE_CHANNEL}[a.gate]
                 e.m_scale = a.scale
                 e.m_unit_norm, e.m_vmix_role, e.m_vmix, e.m_temp_f32 = int(a.unit_norm), lw.get("m_vmix_role", 0), lw.get("m_vmix", 0.0), p(lw.get("m_temp"))
+                e.m_no_qk_norm, e.m_keep_first, e.m_maps, e.m_softcap = int(not a.qk_norm), a.keep_first if a.window else 0, a.maps, a.softcap
+                e.m_lambda, e.m_diff_scale = lw.get("m_lambda", 0.0), 1.0 - a.diff
+                e.m_in_bias_f32, e.m_in_bias = p(lw.get("m_in_bias")), p(lw.get("m_in_bias_st"))
                 e.m_in, e.m_qnorm_f32, e.m_knorm_f32, e.m_out = p(lw["m_in"]), p(lw.get("m_qnorm")), p(lw.get("m_knorm")), p(lw["m_out"])
             elif L.type == "mamba2":
                 s = L.ssd
@@ -419,21 +446,22 @@ class SeqLMForCausalLM:
                 e.e_experts, e.e_top, e.e_ff, e.e_shared_ff, e.e_scale = x.experts, x.top, x.ff, x.shared_ff, x.scale
                 e.e_router_kind = {"softmax": _cabi.ROUTER_SOFTMAX, "topk_softmax": _cabi.ROUTER_TOPK_SOFTMAX}.get(x.router, _cabi.ROUTER_SIGMOID)
                 e.e_identity, e.e_groups, e.e_keep, e.e_limit = x.identity, x.groups, x.keep, x.limit
-                e.e_act = {"clamp_glu": _cabi.EXPERT_CLAMP_GLU, "silu_glu": _cabi.EXPERT_SILU_GLU}.get(x.act, _cabi.EXPERT_RELU2)
-                e.e_up_il16 = lw.get("e_up_il16", 0)
+                e.e_act = {"clamp_glu": _cabi.EXPERT_CLAMP_GLU, "silu_glu": _cabi.EXPERT_SILU_GLU, "gelu": _cabi.EXPERT_GELU}.get(x.act, _cabi.EXPERT_RELU2)
+                e.e_up_il16, e.e_group_top, e.e_shared_ungated = lw.get("e_up_il16", 0), x.group_top, int(not x.shared_gate)
                 e.norm2_f32, e.e_router, e.e_correction_f32 = p(lw.get("norm2")), p(lw["e_router"]), p(lw.get("e_correction"))
                 e.e_up, e.e_down = p(lw["e_up"]), p(lw["e_down"])
                 e.e_shared_up, e.e_shared_down = p(lw.get("e_shared_up")), p(lw.get("e_shared_down"))
             elif L.ff:
                 e.ff_kind = _cabi.FF_MLP if cfg.dense == "mlp" else _cabi.FF_GLU
+                e.ff_act = _cabi.ACT_RELU2 if cfg.dense_act == "relu2" else _cabi.ACT_GELU_TANH
                 e.norm2_f32, e.ff_in, e.ff_out = p(lw.get("norm2")), p(lw["ff_in"]), p(lw["ff_out"])
         desc = _cabi.SeqModelDesc(
             width=cfg.width, vocab=cfg.vocab, n_layers=len(cfg.layers),
             dtype=_cabi.DT_F32 if self.dtype == torch.float32 else _cabi.DT_BF16, rows_padded8=1, eps=cfg.eps, alpha=cfg.alpha,
             embed_scale=cfg.embed_scale, logit_softcap=cfg.logit_softcap,
-            block={"prenorm_hc": _cabi.BLOCK_PRENORM_HC, "parallel": _cabi.BLOCK_PARALLEL, "branchnorm": _cabi.BLOCK_BRANCHNORM}.get(cfg.block, _cabi.BLOCK_POSTNORM),
+            block={"prenorm_hc": _cabi.BLOCK_PRENORM_HC, "parallel": _cabi.BLOCK_PARALLEL, "branchnorm": _cabi.BLOCK_BRANCHNORM, "sandwich": _cabi.BLOCK_SANDWICH}.get(cfg.block, _cabi.BLOCK_POSTNORM),
             streams=cfg.streams, canon_taps=cfg.canon_taps,
-            norm_kind=_cabi.NORM_DYT if cfg.norm == "dyt" else _cabi.NORM_RMS, final_norm_alpha=w.final_norm_alpha,
+            norm_kind={"dyt": _cabi.NORM_DYT, "layer": _cabi.NORM_LAYER}.get(cfg.norm, _cabi.NORM_RMS), final_norm_alpha=w.final_norm_alpha,
             logit_scale=cfg.logit_scale, final_norm_bias_f32=p(w.final_norm_bias),
             embed=p(w.embed), inv_freq_f32=p(w.inv_freq),
             final_norm_f32=p(w.final_norm), head=p(w.head), layers=arr)
