@@ -631,7 +631,7 @@ class SeqModelConfig:
             elif L.type in ("retention", "lightning"):
                 t = L.retention
                 if len(t.decay) != t.heads or t.dim > 512 or t.rot.dims % 2 or t.rot.dims > t.dim or \
-                        any(not 0.0 < x <= 1.0 for x in t.decay):
+                        any(not 0.0 <= x <= 1.0 for x in t.decay):
                     raise ValueError(f"layer {i}: unsupported retention sizes {t}")
             elif L.type == "latent_attention":
                 a = L.latent

@@ -715,7 +715,8 @@ __device__ __forceinline__ void stage_bf16_rows(bf16* dst, int n_rows, int ld_ds
 // MAPS = 2 (differential attention; KH = 2): the two groups of warps take the two maps of one head over the SAME key tiles, so a tile's
 // V rows are staged once for both; at the end the second group hands its normalised output to the first, which writes the normed
 // difference. D is a map's width; key rows hold both maps.
-template <bool VEC8, int KH, int NV, int NBUF = 2, int MAPS = 1>
+// EXT: soft-capped scores, kept first positions, key rows of two maps, fp32 output of one map (compiled out of the plain form).
+template <bool VEC8, int KH, int NV, int NBUF = 2, int MAPS = 1, bool EXT = false>
 __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 : 0) attn_chunk_sink_mma_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pages,
                                                                   const bf16* __restrict__ v_pages, const int* __restrict__ page_table,
                                                                   int page_size, const bf16* __restrict__ gate, int ld_gate,
@@ -727,7 +728,7 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 :
     // NV output tiles of 128 channels per CTA (NV = 2: values of up to 256 channels against one pass over the scores)
     constexpr int MVW = 128 * NV, MLV = MVW + 8;
     const int Dp = (D + 15) / 16 * 16, LQ = Dp + 8;
-    static_assert(MAPS == 1 || KH == 2, "one group of warps per map");
+    static_assert(MAPS == 1 || (KH == 2 && EXT), "one group of warps per map");
     bf16* sQ = reinterpret_cast<bf16*>(smem_attn);     // [MAPS][MQ][LQ]
     constexpr int KT = MAPS == 2 ? MK : KH * MK;        // keys per step of the CTA: one 64-key tile per group of 4 warps (two maps: one for both)
     constexpr int KR = MAPS * KT;                       // K rows of a buffer (the second map's tile behind the first's)
@@ -739,10 +740,10 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 :
     const int rows = min(MQ, S - t0);
     const int pf = past + t0, pl = pf + rows - 1;
     const int kbeg = first_key(pf, chunk, opt.window);       // the first row's first key: no later row starts earlier
-    const int keep = min(opt.keep_first, kbeg), k_start = keep > 0 ? 0 : kbeg;
+    const int keep_first = EXT ? opt.keep_first : 0, keep = min(keep_first, kbeg), k_start = keep > 0 ? 0 : kbeg;
     // a CTA of one map works on head h = head * opt.maps + map (its K columns start at map * D), a CTA of both maps on head h
-    const int ld_k = D * opt.maps, koff = MAPS == 1 ? (h % opt.maps) * D : 0;
-    const float inv_cap = opt.softcap > 0.f ? 1.f / opt.softcap : 0.f;
+    const int ld_k = EXT ? D * opt.maps : D, koff = EXT && MAPS == 1 ? (h % opt.maps) * D : 0;
+    const float inv_cap = EXT && opt.softcap > 0.f ? 1.f / opt.softcap : 0.f;
     const int dvv = min(MVW, DV - c0), DVp = (dvv + 15) / 16 * 16;
     const int warp = (threadIdx.x >> 5) & 3, kh = threadIdx.x >> 7, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
     // queries: fp32 -> bf16, zero padding
@@ -774,7 +775,7 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 :
         const int kpr = Dp / 8, kpm = MAPS * kpr, vpr = DVp / 8, nw = blockDim.x >> 5, wid = threadIdx.x >> 5;
         int pj = k0 + wid, pg = pj / page_size, slot = pj - pg * page_size;
         for (int r = wid; r < KT; r += nw) {
-            const bool row_ok = pj <= pl && (pj >= kbeg || pj < keep);
+            const bool row_ok = pj <= pl && (!EXT || pj >= kbeg || pj < keep);
             const size_t ro = row_ok ? ((size_t)page_table[pg] * G + g) * page_size + slot : 0;
             for (int cu = lane; cu < kpm + vpr; cu += 32) {
                 if (cu < kpm) {
@@ -825,7 +826,7 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 :
             __syncthreads();
         }
         // no visible key for this group in this step (barriers are above)
-        if (k0 > pl || (k0 >= keep && k0 + MK <= kbeg)) continue;
+        if (k0 > pl || (EXT && k0 >= keep && k0 + MK <= kbeg)) continue;
         const bf16* sQm = sQ + (size_t)(MAPS == 2 ? kh : 0) * MQ * LQ;
         float sc[8][4] = {};
         for (int ks = 0; ks < Dp; ks += 16) {
@@ -843,7 +844,7 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 :
         // A tile every row of the CTA sees in full (at or after the last row's chunk start, wholly before the first row)
         // skips the mask. The exponentials are exp2 of pre-scaled arguments: their error (2^-22) is far below the bf16
         // rounding of the weights that follows.
-        const bool full = k0 + MK - 1 <= pf && rows == MQ && (k0 >= first_key(pl, chunk, opt.window) || k0 + MK <= opt.keep_first);
+        const bool full = k0 + MK - 1 <= pf && rows == MQ && (k0 >= first_key(pl, chunk, opt.window) || (EXT && k0 + MK <= keep_first));
         float corr[2];
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
@@ -853,10 +854,10 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 :
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     float v = sc[j][2 * i + e] * scale;
-                    if (opt.softcap > 0.f) v = soft_cap_fast(v, opt.softcap, inv_cap);
+                    if (EXT && opt.softcap > 0.f) v = soft_cap_fast(v, opt.softcap, inv_cap);
                     if (!full) {
                         const int pj = k0 + j * 8 + 2 * tq + e;
-                        const bool ok = pj <= p_row[i] && (pj >= lo_row[i] || pj < opt.keep_first) && r_lo + 8 * i < rows;
+                        const bool ok = pj <= p_row[i] && (pj >= lo_row[i] || (EXT && pj < keep_first)) && r_lo + 8 * i < rows;
                         v = ok ? v : -INFINITY;
                     }
                     sc[j][2 * i + e] = v;
@@ -999,7 +1000,7 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 :
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int col = nt * 8 + 2 * tq + e;
-                if (col < dvv && opt.raw) {
+                if (EXT && col < dvv && opt.raw) {
                     opt.raw[((size_t)t * Hq + h) * DV + c0 + col] = o[nt][2 * i + e] * f;
                 } else if (col < dvv) {
                     const float gv = (gate && opt.gate_channel) ? gate_of(gate, ld_gate, t, h, c0 + col, DV, true) : 1.f;
@@ -1012,7 +1013,8 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 :
 int launch_attn_mma(const float* q, const void* k_pages, const void* v_pages, const int* page_table, int page_size,
                     const void* gate, int ld_gate, void* out, int ld_out, int S, int Hq, int G, int D, int DV, int chunk,
                     float scale, SeqPos pos, cudaStream_t s, const float* sink, int ld_v, AttnOpts opt) {
-    static SmemAttrOnce once82, once82s, once81, once1, once81w, once1w;
+    static SmemAttrOnce once82, once82s, once81, once1, once81w, once1w, once81x, once1x, once81wx, once1wx;
+    const bool ext = opt.softcap > 0.f || opt.keep_first > 0 || opt.maps > 1;
     // two groups of warps: one K/V buffer and two CTAs per SM (default), or two buffers and one CTA (LIVECC_B200_SEQ_ATTN_NBUF=2)
     static const int nbuf2 = [] { const char* e = getenv("LIVECC_B200_SEQ_ATTN_NBUF"); return e ? atoi(e) : 1; }();
     const int Dp = (D + 15) / 16 * 16;
@@ -1022,7 +1024,7 @@ int launch_attn_mma(const float* q, const void* k_pages, const void* v_pages, co
     // merge (68 floats per thread of a group, 34 KB) lies over the K and V buffers, whose V part alone is 68 KB
     // values wider than 128 channels: two output tiles per CTA against one pass over the scores (one group of warps)
     const bool wide = DV > 128;
-    const bool two = vec8 && Dp <= 128 && !wide;
+    const bool two = vec8 && Dp <= 128 && !wide && !ext;
     const int nbuf = vec8 ? ((two && nbuf2 == 1) ? 1 : 2) : 1, kh = two ? 2 : 1, MVW = wide ? 256 : 128, MLV = MVW + 8;
     auto bytes = [&](int dp) { return ((size_t)MQ * (dp + 8) + (size_t)nbuf * kh * MK * (dp + 8 + MLV)) * sizeof(bf16); };
     const size_t smem = bytes(Dp), smem_max = bytes(two ? 128 : kAttnMmaMaxDim);
@@ -1035,7 +1037,11 @@ int launch_attn_mma(const float* q, const void* k_pages, const void* v_pages, co
                                                                            page_size, (const bf16*)gate, ld_gate, (bf16*)out, ld_out, \
                                                                            S, Hq, G, D, DV, chunk, scale, pos, sink, ld_v, opt);  \
     } while (0)
-    if (two && nbuf == 1) LCC_ATTN_MMA(once82s, true, 2, 1, 1);
+    if (ext && wide && vec8) LCC_ATTN_MMA(once81wx, true, 1, 2, 2, 1, true);
+    else if (ext && wide) LCC_ATTN_MMA(once1wx, false, 1, 2, 2, 1, true);
+    else if (ext && vec8) LCC_ATTN_MMA(once81x, true, 1, 1, 2, 1, true);
+    else if (ext) LCC_ATTN_MMA(once1x, false, 1, 1, 2, 1, true);
+    else if (two && nbuf == 1) LCC_ATTN_MMA(once82s, true, 2, 1, 1);
     else if (two) LCC_ATTN_MMA(once82, true, 2, 1);
     else if (wide && vec8) LCC_ATTN_MMA(once81w, true, 1, 2);
     else if (wide) LCC_ATTN_MMA(once1w, false, 1, 2);
@@ -1064,8 +1070,8 @@ int launch_attn_mma_maps(const float* q, const void* k_pages, const void* v_page
     count_launch();
 #define LCC_ATTN_MAPS(ONCE, VEC, NVN, NB)                                                                                        \
     do {                                                                                                                         \
-        if (ensure_dyn_smem(ONCE, attn_chunk_sink_mma_kernel<VEC, 2, NVN, NB, 2>, (int)smem_max)) return -100;                   \
-        attn_chunk_sink_mma_kernel<VEC, 2, NVN, NB, 2><<<grid, 256, smem, s>>>(q, (const bf16*)k_pages, (const bf16*)v_pages, page_table, page_size, \
+        if (ensure_dyn_smem(ONCE, attn_chunk_sink_mma_kernel<VEC, 2, NVN, NB, 2, true>, (int)smem_max)) return -100;                   \
+        attn_chunk_sink_mma_kernel<VEC, 2, NVN, NB, 2, true><<<grid, 256, smem, s>>>(q, (const bf16*)k_pages, (const bf16*)v_pages, page_table, page_size, \
                                                                                nullptr, 0, (bf16*)out, ld_out, S, Hq, G, D, DV, chunk, scale, pos, \
                                                                                sink, ld_v, opt);                                 \
     } while (0)

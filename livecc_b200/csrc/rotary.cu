@@ -13,6 +13,16 @@ template <typename T> __device__ __forceinline__ float ldf(const T* p);
 template <> __device__ __forceinline__ float ldf<float>(const float* p) { return *p; }
 template <> __device__ __forceinline__ float ldf<bf16>(const bf16* p) { return __bfloat162float(*p); }
 
+__device__ __forceinline__ void ld4(const float* p, float (&v)[4]) {
+    const float4 u = *reinterpret_cast<const float4*>(p);
+    v[0] = u.x; v[1] = u.y; v[2] = u.z; v[3] = u.w;
+}
+__device__ __forceinline__ void ld4(const bf16* p, float (&v)[4]) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+
 __device__ __forceinline__ int seq_past(const SeqPos& p) { return p.kv_len ? *p.kv_len : p.past; }
 __device__ __forceinline__ bool seq_done(const SeqPos& p) { return p.finished && *p.finished; }
 
@@ -20,7 +30,7 @@ struct Segs { RotarySegment s[4]; int n; };
 
 // gridDim.y CTAs per row (several when the call has few rows, so that a decode step's single row is not one CTA's serial
 // walk); together their threads walk the output channels of every segment.
-template <typename T>
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) rotary_pack_kernel(const T* __restrict__ in, int ld_in, float* __restrict__ out, int ld_out,
                                                           Segs segs, const float* __restrict__ inv_freq, float mag,
                                                           const float* __restrict__ fill, float* __restrict__ fill_out, int fill_n,
@@ -33,6 +43,16 @@ __global__ void __launch_bounds__(256) rotary_pack_kernel(const T* __restrict__ 
     for (int si = 0; si < segs.n; ++si) {
         const RotarySegment sg = segs.s[si];
         const int n = sg.heads * sg.dim, half = sg.rot_dims / 2;
+        if (VEC && sg.rot_dims == 0) {       // nothing turns: four neighbouring channels per thread
+            for (int i = (threadIdx.x + blockIdx.y * blockDim.x) * 4; i < n; i += blockDim.x * gridDim.y * 4) {
+                float v[4];
+                ld4(row + sg.col_in + i, v);
+#pragma unroll
+                for (int u = 0; u < 4; ++u) v[u] = (sg.silu ? v[u] / (1.f + expf(-v[u])) : v[u]) * sg.scale;
+                *reinterpret_cast<float4*>(orow + sg.col_out + i) = make_float4(v[0], v[1], v[2], v[3]);
+            }
+            continue;
+        }
         for (int i = threadIdx.x + blockIdx.y * blockDim.x; i < n; i += blockDim.x * gridDim.y) {
             const int d = i % sg.dim, hb = i - d;
             const int r = d - sg.rot_off;
@@ -69,10 +89,18 @@ int rotary_pack_f32(int dt, const void* in, int ld_in, float* out, int ld_out, c
     }
     count_launch();
     const dim3 S_grid(S, S < 32 ? 8 : 1);
-    if (dt == DT_F32)
-        rotary_pack_kernel<float><<<S_grid, 256, 0, s>>>((const float*)in, ld_in, out, ld_out, g, inv_freq, mag, fill, fill_out, fill_n, pos);
-    else
-        rotary_pack_kernel<bf16><<<S_grid, 256, 0, s>>>((const bf16*)in, ld_in, out, ld_out, g, inv_freq, mag, fill, fill_out, fill_n, pos);
+    // four channels per thread in segments without a rotation, when every row and segment starts on a whole group
+    bool vec = (ld_in % 4) == 0 && (ld_out % 4) == 0 && ((uintptr_t)in % (4 * dt_size(dt))) == 0 && ((uintptr_t)out % 16) == 0;
+    bool any = false;
+    for (int i = 0; i < n_seg; ++i) {
+        vec = vec && (seg[i].col_in % 4) == 0 && (seg[i].col_out % 4) == 0 && (seg[i].heads * seg[i].dim) % 4 == 0;
+        any = any || seg[i].rot_dims == 0;
+    }
+    vec = vec && any;
+#define LCC_PACK(T, V) rotary_pack_kernel<T, V><<<S_grid, 256, 0, s>>>((const T*)in, ld_in, out, ld_out, g, inv_freq, mag, fill, fill_out, fill_n, pos)
+    if (dt == DT_F32) { if (vec) LCC_PACK(float, true); else LCC_PACK(float, false); }
+    else { if (vec) LCC_PACK(bf16, true); else LCC_PACK(bf16, false); }
+#undef LCC_PACK
     return cudaGetLastError() == cudaSuccess ? 0 : -100;
 }
 

@@ -108,6 +108,27 @@ def lugizen_config(width: int, n_layers: int, ff: int, window: int, vocab: int =
                                      "canon": {"taps": 4}})
 
 
+def kapitar_config(width: int, n_layers: int, ff: int, window: int, vocab: int = 32768) -> SeqModelConfig:
+    """Norms on either side of every sublayer; layers in the pattern differential attention, differential attention, lightning
+    attention, differential attention. Differential attention: width/256 heads of two 128-channel maps over 256-channel values (8
+    query heads per key/value head), scores capped at 50, a window of `window` positions that keeps the first 16. Lightning
+    attention: width/128 heads of 128 key and 128 value channels, decays 1 - 2^-(5+h). The first layer has a two-matrix feed-forward
+    of width 3 ff / 2, every other layer 16 two-matrix experts of width ff/4, 4 per token out of the best 3 of 4 groups, beside a
+    shared expert of width ff/2: every token reads 3 x width x ff feed-forward weights, the dense gated `ff` of the models beside it."""
+    heads, layers = width // 256, []
+    att = dict(heads=heads, kv_heads=max(1, heads // 8), dim=128, vdim=256, mask={"size": window, "keep_first": 16}, scale=128 ** -0.5,
+               softcap=50.0, diff=0.6)
+    rh = width // 128
+    light = dict(heads=rh, dim=128, vdim=128, decay=[1.0 - 2.0 ** (-5 - (h % 8)) for h in range(rh)])
+    moe = {"kind": "moe", "expert": {"ff": ff // 4 // 8 * 8}, "router": {"experts": 16, "top": 4, "groups": {"count": 4, "keep": 3}},
+           "shared": {"ff": ff // 2 // 8 * 8}}
+    for i in range(n_layers):
+        L = {"type": "lightning", "mixer": light} if i % 4 == 2 else {"type": "attention", "mixer": att}
+        L["mlp"] = {"kind": "dense", "ff": 3 * ff // 2 // 8 * 8} if i == 0 else moe
+        layers.append(L)
+    return SeqModelConfig.from_json({"architecture": "Kapitar", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": 1e-6}})
+
+
 def qwen_config(width: int, n_layers: int, ff: int, vocab: int = 32768) -> LiveCCConfig:
     heads = width // 128
     return LiveCCConfig(
@@ -158,7 +179,9 @@ def time_qwen(model, prompt_len: int, new_tokens: int, steps: int, warmup: int) 
 def active_weight_bytes(model) -> int:
     """Bytes of weights one decode step reads: everything but the embedding table (one row is read) and, in a routed
     feed-forward, the experts that were not chosen."""
-    n = model.weights.nbytes() - model.weights.embed.numel() * model.weights.embed.element_size()
+    n = model.weights.nbytes()
+    if not model.config.tied_head:       # (a tied head reads the whole table)
+        n -= model.weights.embed.numel() * model.weights.embed.element_size()
     for L, w in zip(model.config.layers, model.weights.layers):
         if L.moe:
             per = (w["e_up"].numel() + w["e_down"].numel()) * w["e_up"].element_size() // L.moe.experts
@@ -176,9 +199,10 @@ def run(sizes: List[str], prompt_lens: List[int], new_tokens: int, steps: int, w
         width, n_layers, ff, chunk = SIZES[name]
         rec = {}
         arms = {"Bimopel": ["bimopel"], "Kedelorn": ["kedelorn", "bimopel"], "Dibedra": ["dibedra", "kedelorn"],
-                "Lugizen": ["lugizen", "kedelorn"]}[design]
+                "Lugizen": ["lugizen", "kedelorn"], "Kapitar": ["kapitar", "dibedra", "kedelorn"]}[design]
         make = {"bimopel": lambda: seq_config(width, n_layers, ff, chunk), "kedelorn": lambda: kedelorn_config(width, n_layers, ff),
-                "dibedra": lambda: dibedra_config(width, n_layers, ff, chunk), "lugizen": lambda: lugizen_config(width, n_layers, ff, chunk)}
+                "dibedra": lambda: dibedra_config(width, n_layers, ff, chunk), "lugizen": lambda: lugizen_config(width, n_layers, ff, chunk),
+                "kapitar": lambda: kapitar_config(width, n_layers, ff, chunk)}
         for label, cfg in [(a, make[a]()) for a in arms]:
             m = SeqLMForCausalLM.from_state_dict(cfg, synthetic_seq_tensors(cfg, seed=7, device="cuda"), dtype,
                                                  max_tokens=max(prompt_lens) + new_tokens + 64)
@@ -201,7 +225,7 @@ def run(sizes: List[str], prompt_lens: List[int], new_tokens: int, steps: int, w
 
 
 def main(args, design: str = "Bimopel") -> Dict:
-    """bench.py --arch seq | kedelorn | dibedra | lugizen: one JSON line; `value` = decode tokens/s of the first size at the first prompt length."""
+    """bench.py --arch seq | kedelorn | dibedra | lugizen | kapitar: one JSON line; `value` = decode tokens/s of the first size at the first prompt length."""
     sizes = [s for s in (args.seq_sizes.split(",") if args.seq_sizes else list(SIZES)) if s in SIZES]
     lens = [int(x) for x in args.seq_prompt.split(",")]
     res = run(sizes, lens, args.max_new_tokens if args.max_new_tokens > 16 else 64, args.steps, max(args.warmup, 3), design=design)
@@ -209,7 +233,7 @@ def main(args, design: str = "Bimopel") -> Dict:
     return {"metric": "decode_tokens_per_s", "value": first["decode_tok_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
             "warmup": max(args.warmup, 3), "ms_per_step": first["decode_ms_per_token"], "higher_is_better": True, "dtype": "bf16",
             "data": "synthetic (random weights, random ids)", "vs_baseline": None,
-            "config": {"model": f"{design} {sizes[0]} beside " + {"Kedelorn": "Bimopel and the ", "Dibedra": "Kedelorn and the ", "Lugizen": "Kedelorn and the "}.get(design, "") +
+            "config": {"model": f"{design} {sizes[0]} beside " + {"Kedelorn": "Bimopel and the ", "Dibedra": "Kedelorn and the ", "Lugizen": "Kedelorn and the ", "Kapitar": "Dibedra, Kedelorn and the "}.get(design, "") +
                                 "Qwen2-style decoder of equal width/depth/ff", "global_batch": 1,
                        "seq_len": lens[0], "parallelism": "1 gpu", "l2": "weights of every size exceed L2"},
             "sizes": res}

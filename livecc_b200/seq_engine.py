@@ -154,7 +154,7 @@ class SeqWeights:
                 check(m + "v", (rt.heads * rt.vdim, W)), check(m + "g", (rt.heads * rt.vdim, W)), check(m + "o", (W, rt.heads * rt.vdim))
                 w["t_in"] = mat(m + "q", m + "k", m + "v", m + "g")
                 w["t_out"] = mat(m + "o")
-                w["t_log_decay"] = torch.log(torch.tensor(rt.decay, dtype=torch.float64)).to(torch.float32).to(device)
+                w["t_log_decay"] = torch.log(torch.tensor(rt.decay, dtype=torch.float64).clamp_min(1e-35)).to(torch.float32).to(device)
                 if rt.whole_norm:
                     check(m + "norm", (rt.heads * rt.vdim,))
                     w["t_norm"] = f32(get(m + "norm"))
