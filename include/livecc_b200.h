@@ -31,7 +31,7 @@
 extern "C" {
 #endif
 
-#define LCC_ABI_VERSION 12
+#define LCC_ABI_VERSION 13
 #define LCC_PAGE_SIZE 64
 
 typedef struct lcc_ctx lcc_ctx;
@@ -293,7 +293,8 @@ int lcc_resize_bicubic_aa_u8(lcc_ctx* ctx, const lcc_resize_plan* plan, const ui
 
 /* ---- hybrid sequence models: decoder-only language models whose layers mix tokens with a state-space recurrence, gated
  * linear attention, retention, a gated delta rule, chunk-local attention, latent attention or sliding-window attention. A layer is
- *     x <- norm1(alpha * x + mixer(x)),  then (if it has a feed-forward)  x <- norm2(alpha * x + ff(x))       (post-norm)
+ *     x <- norm1(alpha * x + ls1 * mixer(x)),  then (if it has a feed-forward)  x <- norm2(alpha * x + ls2 * ff(x))   (post-norm; the
+ * vectors ls1, ls2 are optional)
  * or, in a model with LCC_BLOCK_PRENORM_HC, pre-norm sublayers on several residual streams (see LCC_BLOCK_PRENORM_HC),
  * or, with LCC_BLOCK_PARALLEL, x <- x + mixer(norm1(x)) + ff(norm1(x)),
  * or, with LCC_BLOCK_BRANCHNORM, x <- x + norm1(mixer(x + canon(x))), then x <- x + norm2(ff(x)) (the norm sits on the sublayer's
@@ -311,17 +312,19 @@ int lcc_resize_bicubic_aa_u8(lcc_ctx* ctx, const lcc_resize_plan* plan, const ui
 #define LCC_MIX_LATENT 4    /* causal softmax attention over a cached low-rank latent + one shared rotary key part, per-head sink and sigmoid gate */
 #define LCC_MIX_ATTENTION 5 /* softmax attention over paged K/V: per-head q/k RMS norm, rotary positions on part of a head, a sliding
                                window (which may keep the first positions) and / or chunks, optional sink, values projected or taken
-                               from the keys as projected, output gate per head or per channel, soft-capped scores, two maps per head
+                               from the keys as projected, output gate per head or per channel, soft-capped scores, a learned bias per
+                               distance, queries scaled with their position, keys and values of another layer, two maps per head
                                whose normed difference is the output (every option a field of the layer) */
 #define LCC_MIX_DELTA 6     /* gated delta rule with a decay per key channel: q/k/v through a short causal convolution + silu, unit-length q
                                and k, S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; unit-rms heads x weight x sigmoid
                                gate -> out-proj (decays and output gate come through low-rank bottlenecks) */
-#define LCC_FF_GLU 0        /* dense gated feed-forward: gelu_tanh(gate) * up */
+#define LCC_FF_GLU 0        /* dense gated feed-forward: gelu_tanh(gate) * up, or with LCC_ACT_CLAMP_GLU the clamped form */
 #define LCC_FF_MOE 1        /* routed experts (sigmoid or softmax router, top-k of score + correction, optionally inside the best groups
                                of neighbouring experts; relu^2 or clamped gated experts; identity experts) + gated shared expert */
 #define LCC_FF_MLP 2        /* dense two-matrix feed-forward: down(act(up x)), act LCC_ACT_* */
 #define LCC_ACT_GELU_TANH 0
 #define LCC_ACT_RELU2 1     /* relu(z)^2 */
+#define LCC_ACT_CLAMP_GLU 2 /* LCC_FF_GLU: g = min(gate, limit), u = clamp(up, +-limit); g * sigmoid(1.702 g) * (u + 1) */
 #define LCC_BLOCK_POSTNORM 0 /* x <- norm(alpha * x + sublayer(x)) */
 #define LCC_BLOCK_PRENORM_HC 1 /* `streams` residual streams x_s; per sublayer: u = sum_s in[s] x_s; y = sublayer(norm(u));
                                   x_t <- sum_s mix[s][t] x_s + out[t] y. The model's output is the sum of the streams. */
@@ -365,9 +368,11 @@ typedef struct {
     int32_t a_heads, a_dim, a_rot_dim, a_vdim, a_rank, a_kv_from;
     float a_scale;
     /* a_q_rank > 0: the queries come through a latent of that many channels (a_in rows [q latent | latent, key part | gate], RMS norm
-     * with a_q_norm_f32, then a_uq); a_window > 0: a row at position i sees j with i - j < a_window; a_gate: a_in ends with one gate
-     * row per head; a_sink_f32 NULL: ordinary softmax */
-    int32_t a_q_rank, a_window, a_gate;
+     * with a_q_norm_f32, then a_uq); a_window > 0: a row at position i sees j with i - j < a_window; a_gate LCC_GATE_*: a_in ends with one
+     * gate row per head, or (LCC_GATE_CHANNEL: applied behind the value up-projection) with heads * vdim gate rows whose block starts
+     * at a multiple of 8; a_rot_pairs: channel 2i of the rotated part turns with 2i+1, else i with i + rot_dim/2; a_sink_f32 NULL:
+     * ordinary softmax */
+    int32_t a_q_rank, a_window, a_gate, a_rot_pairs;
     float rot_mag;  /* factor on cos and sin of the rotation (1 without long-context scaling) */
     /* LCC_MIX_ATTENTION: m_heads query heads over m_kv_heads key/value heads; per-head RMS norm of q and k (weights [m_dim], shared by
      * the heads); the first m_rot_dims channels of a head rotated (m_rot_pairs: channel 2i with 2i+1, else i with i + dims/2);
@@ -387,12 +392,20 @@ typedef struct {
      * times m_diff_scale (m_in rows [q: Hq*2*dim | k: G*2*dim | v], K pages [page][G][page_size][2*dim]) */
     int32_t m_no_qk_norm, m_keep_first, m_maps;
     float m_softcap, m_lambda, m_diff_scale;
+    /* m_kv_from >= 0: the layer projects queries only and reads that earlier layer's keys and values (m_in rows [q | gate]; its own mask);
+     * m_temp_every > 0: the queries at position p are multiplied by 1 + m_temp_coef * ln(floor((p + 1) / m_temp_every) + 1);
+     * m_bias_f32 [heads][m_bias_len]: added to a score behind scale and cap, entry d for a key d positions back (the last entry for
+     * every key further away); NULL: none */
+    int32_t m_kv_from, m_temp_every, m_bias_len;
+    float m_temp_coef;
     /* LCC_MIX_DELTA: d_heads value heads of d_vdim channels over d_kv_heads query/key heads of d_dim channels, d_conv taps, bottleneck
      * ranks of the decay and of the output gate */
     int32_t d_heads, d_kv_heads, d_dim, d_vdim, d_conv, d_rank_a, d_rank_g;
     /* feed-forward: ff_kind LCC_FF_*; MoE: e_experts experts of width e_ff, e_top per token, weights = score * e_scale,
      * shared expert of width e_shared_ff (0 = none) */
-    int32_t ff_act;    /* LCC_FF_MLP: LCC_ACT_* */
+    int32_t ff_act;    /* LCC_ACT_* (LCC_FF_MLP: gelu or relu^2; LCC_FF_GLU: gelu or the clamped form) */
+    int32_t ff_il16;   /* LCC_ACT_CLAMP_GLU: gate and up rows of ff_in interleaved in groups of 16 (as e_up_il16) */
+    float ff_limit;    /* LCC_ACT_CLAMP_GLU: its clamp */
     int32_t ff_kind, e_experts, e_top, e_ff, e_shared_ff;
     float e_scale;
     /* e_router_kind LCC_ROUTER_*; the last e_identity router outputs (beyond the e_experts real ones) stand for experts that return
@@ -408,6 +421,9 @@ typedef struct {
     /* weights: matrices [out, in] in the model's storage type; everything named *_f32 is fp32 */
     const float *norm1_f32, *norm2_f32;
     const float *norm1b_f32, *norm2b_f32; /* LCC_BLOCK_SANDWICH: the norms behind the sublayers */
+    const float *ls1_f32, *ls2_f32;       /* LCC_BLOCK_POSTNORM: [width] factors on the sublayers' outputs (NULL: none) */
+    const float* m_bias_f32;              /* [m_heads][m_bias_len] or NULL */
+    const float* e_router_bias_f32;       /* [experts + identity]: added to the router's logits themselves (NULL: zeros) */
     const float* m_in_bias_f32;  /* biases of the q, k, v rows of m_in (NULL: none) */
     const void* m_in_bias;       /* optional copy in the storage type, padded like the matrix rows (tensor-core epilogue) */
     const float* canon_w_f32;  /* LCC_BLOCK_BRANCHNORM: [width, canon_taps] taps of the convolution in front of the mixer (NULL: none) */
@@ -423,7 +439,7 @@ typedef struct {
     const float* d_norm_f32;   /* [vdim], shared by the heads */
     const void* d_out;         /* [width, heads*vdim] */
     const float* norm1_bias_f32; /* LCC_NORM_DYT: [width] */
-    const void* m_in;          /* [Hq*dim + G*dim (+ G*vdim) + gate rows, width], rows [q | k | (v) | gate] */
+    const void* m_in;          /* [Hq*dim + G*dim (+ G*vdim) + gate rows, width], rows [q | k | (v) | gate]; m_kv_from >= 0: [q | gate] */
     const float *m_qnorm_f32, *m_knorm_f32; /* [dim] each */
     const void* m_out;         /* [width, Hq*vdim] */
     const void* s_in;          /* [2*inner + 2*groups*state + heads, width], rows [z | x | B | C | dt] */
@@ -442,7 +458,7 @@ typedef struct {
     const float* r_norm_f32;   /* [vdim], shared by the heads */
     const void* r_out;         /* [width, heads*vdim] */
     const float* r_branch_norm_f32; /* [width] */
-    const void* ff_in;         /* LCC_FF_GLU: [2*ff, width], rows [gate | up]; act = gelu_tanh(gate) * up. LCC_FF_MLP: [ff, width] */
+    const void* ff_in;         /* LCC_FF_GLU: [2*ff, width], rows [gate | up] (ff_il16: interleaved). LCC_FF_MLP: [ff, width] */
     const void* ff_out;        /* [width, ff] */
     const float* rot_inv_freq_f32; /* [rot dims / 2]: rotation frequencies of this layer's mixer, computed by the host */
     const void* t_in;          /* [2*heads*dim + 2*heads*vdim, width], rows [q | k | v | gate] */

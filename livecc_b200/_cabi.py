@@ -13,7 +13,7 @@ PKG_DIR = Path(__file__).resolve().parent
 LIB_PATH = PKG_DIR / "liblivecc_sm100a.so"
 HEADER_PATH = PKG_DIR.parent / "include" / "livecc_b200.h"
 
-ABI_VERSION = 12
+ABI_VERSION = 13
 PAGE_SIZE = 64
 
 # epilogue codes (LCC_EPI_*)
@@ -72,17 +72,19 @@ class SeqLayer(C.Structure):
                [("r_tau", C.c_float)] + \
                [(n, C.c_int32) for n in ("t_heads", "t_dim", "t_vdim", "t_rot_dims", "t_silu", "t_plain_keys", "t_whole_norm", "t_gate_sigmoid", "a_heads", "a_dim", "a_rot_dim", "a_vdim",
                                          "a_rank", "a_kv_from")] + [("a_scale", C.c_float)] + \
-               [(n, C.c_int32) for n in ("a_q_rank", "a_window", "a_gate")] + [("rot_mag", C.c_float)] + \
+               [(n, C.c_int32) for n in ("a_q_rank", "a_window", "a_gate", "a_rot_pairs")] + [("rot_mag", C.c_float)] + \
                [(n, C.c_int32) for n in ("m_heads", "m_kv_heads", "m_dim", "m_vdim", "m_window", "m_chunk", "m_rot_dims", "m_rot_pairs",
                                          "m_sink", "m_value_keys", "m_gate")] + [("m_scale", C.c_float)] + \
                [(n, C.c_int32) for n in ("m_unit_norm", "m_vmix_role")] + [("m_vmix", C.c_float)] + \
                [(n, C.c_int32) for n in ("m_no_qk_norm", "m_keep_first", "m_maps")] + \
                [(n, C.c_float) for n in ("m_softcap", "m_lambda", "m_diff_scale")] + \
+               [(n, C.c_int32) for n in ("m_kv_from", "m_temp_every", "m_bias_len")] + [("m_temp_coef", C.c_float)] + \
                [(n, C.c_int32) for n in ("d_heads", "d_kv_heads", "d_dim", "d_vdim", "d_conv", "d_rank_a", "d_rank_g")] + \
-               [(n, C.c_int32) for n in ("ff_act", "ff_kind", "e_experts", "e_top", "e_ff", "e_shared_ff")] + [("e_scale", C.c_float)] + \
+               [("ff_act", C.c_int32), ("ff_il16", C.c_int32), ("ff_limit", C.c_float)] + \
+               [(n, C.c_int32) for n in ("ff_kind", "e_experts", "e_top", "e_ff", "e_shared_ff")] + [("e_scale", C.c_float)] + \
                [(n, C.c_int32) for n in ("e_router_kind", "e_identity", "e_groups", "e_keep", "e_act", "e_group_top", "e_shared_ungated", "e_up_il16")] + \
                [("e_limit", C.c_float), ("norm1_alpha", C.c_float)] + \
-               [(n, C.c_void_p) for n in ("norm1_f32", "norm2_f32", "norm1b_f32", "norm2b_f32", "m_in_bias_f32", "m_in_bias", "canon_w_f32", "m_temp_f32", "a_uq", "a_q_norm_f32", "d_in",
+               [(n, C.c_void_p) for n in ("norm1_f32", "norm2_f32", "norm1b_f32", "norm2b_f32", "ls1_f32", "ls2_f32", "m_bias_f32", "e_router_bias_f32", "m_in_bias_f32", "m_in_bias", "canon_w_f32", "m_temp_f32", "a_uq", "a_q_norm_f32", "d_in",
                                           "d_conv_w_f32", "d_a_up", "d_dt_bias_f32", "d_a_log_f32", "d_g_up", "d_norm_f32", "d_out",
                                           "norm1_bias_f32", "m_in", "m_qnorm_f32", "m_knorm_f32", "m_out", "s_in", "s_conv_w_f32", "s_conv_b_f32", "s_dt_bias_f32",
                                           "s_a_log_f32", "s_skip_f32", "s_norm_f32", "s_out", "l_in", "l_in_bias_f32", "l_in_bias",
@@ -116,7 +118,7 @@ MIX_SSD, MIX_PARALLEL, MIX_RETENTION, MIX_LATENT, MIX_ATTENTION, MIX_DELTA = 1, 
 FF_GLU, FF_MOE, FF_MLP = 0, 1, 2
 BLOCK_POSTNORM, BLOCK_PRENORM_HC, BLOCK_PARALLEL, BLOCK_BRANCHNORM, BLOCK_SANDWICH = 0, 1, 2, 3, 4
 NORM_RMS, NORM_DYT, NORM_LAYER = 0, 1, 2
-ACT_GELU_TANH, ACT_RELU2 = 0, 1
+ACT_GELU_TANH, ACT_RELU2, ACT_CLAMP_GLU = 0, 1, 2
 ROUTER_SIGMOID, ROUTER_SOFTMAX, ROUTER_TOPK_SOFTMAX = 0, 1, 2
 EXPERT_RELU2, EXPERT_CLAMP_GLU, EXPERT_SILU_GLU, EXPERT_GELU = 0, 1, 2, 3
 GATE_NONE, GATE_HEAD, GATE_CHANNEL = 0, 1, 2

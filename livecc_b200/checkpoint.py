@@ -337,6 +337,8 @@ def seq_param_specs(cfg) -> List[Tuple[str, Tuple[int, ...], str]]:
             specs.append((p + "norm2", nshape, norm))
         if sandwich:
             specs += [(p + n, nshape, norm) for n in (("norm1b", "norm2b") if (L.ff or L.moe) else ("norm1b",))]
+        if getattr(cfg, "layer_scale", False):
+            specs += [(p + n, (W,), "ls") for n in (("ls1", "ls2") if (L.ff or L.moe) else ("ls1",))]
         if getattr(cfg, "canon_taps", 0):
             specs.append((p + "canon1", (W, cfg.canon_taps), "canon"))
         if hc:
@@ -369,11 +371,16 @@ def seq_param_specs(cfg) -> List[Tuple[str, Tuple[int, ...], str]]:
             if a.sink:
                 specs.append((m + "sink", (a.heads,), "skip"))
             if a.gate:
-                specs.append((m + "g", (a.heads, W), "w"))
+                specs.append((m + "g", (a.gate_rows, W), "w"))
             specs.append((m + "o", (W, a.heads * a.vdim), "w"))
         elif L.type == "attention":
             a, m = L.attn, p + "mix."
-            specs += [(m + "q", (a.heads * a.maps * a.dim, W), "w"), (m + "k", (a.kv_heads * a.maps * a.dim, W), "w")]
+            own_kv = a.kv_from < 0
+            specs.append((m + "q", (a.heads * a.maps * a.dim, W), "w"))
+            if own_kv:
+                specs.append((m + "k", (a.kv_heads * a.maps * a.dim, W), "w"))
+            if a.rel_max:
+                specs.append((m + "rel", (a.rel_rows or 32, a.heads), "rel"))
             if a.bias:
                 specs += [(m + "q.b", (a.heads * a.maps * a.dim,), "b"), (m + "k.b", (a.kv_heads * a.maps * a.dim,), "b")]
                 if not a.value_keys:
@@ -381,12 +388,12 @@ def seq_param_specs(cfg) -> List[Tuple[str, Tuple[int, ...], str]]:
             if a.maps > 1:
                 specs += [(m + n, (a.dim,), "lam") for n in ("lq1", "lk1", "lq2", "lk2")]
             if a.qk_norm and not a.unit_norm:
-                specs += [(m + "q.norm", (a.dim,), "norm"), (m + "k.norm", (a.dim,), "norm")]
+                specs += [(m + n + ".norm", (a.dim,), "norm") for n in (("q", "k") if own_kv else ("q",))]
             if a.temp:
                 specs.append((m + "temp", (a.heads,), "skip"))
             if a.v_mix:
                 specs.append((m + "vmix", (), "mix"))
-            if not a.value_keys:
+            if not a.value_keys and own_kv:
                 specs.append((m + "v", (a.kv_heads * a.vdim, W), "w"))
             if a.gate != "none":
                 specs.append((m + "g", (a.gate_rows, W), "w"))
@@ -417,6 +424,8 @@ def seq_param_specs(cfg) -> List[Tuple[str, Tuple[int, ...], str]]:
                     specs.append((f"{m}e{j}.gate", (e.ff, W), "w"))
                 specs += [(f"{m}e{j}.up", (e.ff, W), "w"), (f"{m}e{j}.down", (W, e.ff), "w")]
             specs.append((m + "router", (e.outputs, W), "w"))
+            if e.router_bias:
+                specs.append((m + "router.b", (e.outputs,), "rb"))
             if e.router != "topk_softmax" and e.correction:
                 specs.append((m + "correction", (e.outputs,), "b"))
             if e.shared_ff:
@@ -461,6 +470,12 @@ def synthetic_seq_tensors(cfg, seed: int = 1234, device="cpu") -> Dict[str, torc
             t = u * 1.5
         elif kind == "canon":
             t = u * 0.8
+        elif kind == "ls":
+            t = 0.8 + 0.8 * u
+        elif kind == "rel":
+            t = u * 4.0
+        elif kind == "rb":
+            t = u * 2.0
         elif kind == "lam":
             t = u * (2.0 / shape[-1] ** 0.5)
         elif kind == "mix":

@@ -250,6 +250,12 @@ class LatentAttnConfig:
     window: int = 0       # > 0: row i sees j with 0 <= i - j < window
     gate: bool = True     # the per-head sigmoid gate
     sink: bool = True     # the per-head sink logit (False: ordinary softmax)
+    gate_channel: bool = False   # the sigmoid gate has one logit per head and value channel (with `gate`)
+    rot_pairs: bool = False      # channel 2i of the rotated part turns with 2i+1 (else i with i + rot_dim/2)
+
+    @property
+    def gate_rows(self) -> int:
+        return 0 if not self.gate else (self.heads * self.vdim if self.gate_channel else self.heads)
 
 
 @dataclass
@@ -263,7 +269,8 @@ class MoeConfig:
     down(g sigmoid(1.702 g) (u + 1))) or "silu_glu" (down(silu(gate x) * (up x))). `router` "topk_softmax": the `top` largest
     logits are chosen and weighted by the softmax over the chosen logits only (no correction tensor). `act` "gelu": down(gelu(up x)),
     the exact (erf) form. `group_top`: a group scores as the sum of that many of its best choice scores. `correction`: the
-    router has a correction tensor. `shared_gate`: the shared expert sits behind its gate (False: it is added as it is)."""
+    router has a correction tensor. `shared_gate`: the shared expert sits behind its gate (False: it is added as it is).
+    `router_bias`: the router has a bias (tensor `router.b`) that is part of its logits."""
     experts: int
     top: int
     ff: int
@@ -278,6 +285,7 @@ class MoeConfig:
     group_top: int = 1
     correction: bool = True
     shared_gate: bool = True
+    router_bias: bool = False
 
     @property
     def outputs(self) -> int:
@@ -296,7 +304,11 @@ class MaskedAttnConfig:
     softcap * tanh(score / softcap). `maps` = 2, differential attention: every query and key head is two maps of `dim` channels,
     each with a softmax of its own over the same values; the second map's output times lambda is subtracted, lambda =
     exp(lq1 . lk1) - exp(lq2 . lk2) + diff, the difference is brought to unit rms per head and multiplied by 1 - diff.
-    `qk_norm` False: q and k as projected. `bias`: q, k and v projections have biases."""
+    `qk_norm` False: q and k as projected. `bias`: q, k and v projections have biases. `rel_max` > 0: a learned bias per head and
+    distance bucket (tensor `rel` [buckets, heads]) is added to the scores behind scale and cap: one bucket per distance in the first
+    half of the table, then buckets that grow geometrically up to `rel_max` positions. `temp_every` > 0: the queries at position
+    p are multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1). `kv_from` >= 0: the layer projects queries only and reads
+    that earlier layer's cached keys and values. `kind`: the layer's type in config.json (a family may have two attention mixers)."""
     heads: int
     kv_heads: int
     dim: int
@@ -317,6 +329,12 @@ class MaskedAttnConfig:
     softcap: float = 0.0
     keep_first: int = 0
     v_mix: bool = False       # the cached values are (1 - vmix) v + vmix v_first, v_first = the first such layer's values of the token
+    rel_max: float = 0.0
+    rel_rows: int = 0         # rows of the bias table; read from the tensor's shape when 0
+    temp_coef: float = 0.0
+    temp_every: int = 0
+    kv_from: int = -1
+    kind: str = "attention"
 
     @property
     def gate_rows(self) -> int:
@@ -350,6 +368,7 @@ class SeqLayerConfig:
     left: ChunkAttnConfig = None
     right: GlaConfig = None
     ff: int = 0                    # 0 = the layer has no dense feed-forward
+    ff_limit: float = 0.0          # clamp of a clamped gated feed-forward
     retention: RetentionConfig = None   # types "retention" and "lightning"
     latent: LatentAttnConfig = None
     moe: MoeConfig = None          # routed feed-forward instead of the dense one
@@ -382,7 +401,19 @@ SEQ_FAMILIES = {
                     expert="gelu", group_top=2, correction=False, shared_gate=False, tied_head=True,
                     attention=dict(rot_pairs=False, value_keys=False, gate="none", sink=False, qk_norm=False, bias=True, maps=2),
                     lightning=dict(silu=True, key_scale=False, whole_norm=True, gate="sigmoid")),
+    # post-norm blocks whose sublayers pass a factor per channel; two attention mixers without rotation that add a learned bias per
+    # distance (unit-rms heads; or weighted q/k norms, a query temperature, optionally another layer's keys and values), latent
+    # attention with latent queries, pair-interleaved rotation and a gate per channel; clamped gated dense feed-forward; squared-relu experts
+    # chosen by biased logit, weighted by the softmax over the chosen logits, beside a gated shared expert; the head is the embedding table
+    "Poresun": dict(block="postnorm", norm_offset=0.0, positions=None, layer_scale=True, dense="clamp_glu", router="topk_softmax", expert="relu2",
+                    router_bias=True, tied_head=True,
+                    attention=dict(rot_pairs=False, value_keys=False, gate="none", sink=False, unit_norm=True),
+                    attention_2=dict(rot_pairs=False, value_keys=False, gate="none", sink=False),
+                    latent=dict(q_latent=True, gate_channel=True, sink=False, rot_pairs=True)),
 }
+
+# config.json layer types that the masked-attention mixer serves (SeqLayerConfig.type "attention")
+ATTENTION_TYPES = ("attention", "attention_2")
 
 
 @dataclass
@@ -402,7 +433,8 @@ class SeqModelConfig:
     canon_taps: int = 0            # taps of the causal convolution over time in front of every mixer (tensor l<i>.canon1 [width, taps])
     norm_scalar: bool = False      # a norm's weight is ONE number (tensors of one element)
     norm: str = "rms"              # "rms" | "dyt" (tanh(alpha x) w + b; tensors <name>, <name>.b, <name>.alpha) | "layer" (mean taken off, no bias)
-    dense: str = "glu"             # dense feed-forward: "glu" (gelu_tanh(gate) * up) | "mlp" (dense_act(up))
+    dense: str = "glu"             # dense feed-forward: "glu" (gelu_tanh(gate) * up) | "mlp" (dense_act(up)) | "clamp_glu" (MoeConfig.act)
+    layer_scale: bool = False      # post-norm blocks: a factor per channel on every sublayer's output (tensors l<i>.ls1, l<i>.ls2)
     dense_act: str = "gelu_tanh"   # activation of a two-matrix feed-forward: "gelu_tanh" | "relu2"
     tied_head: bool = False        # the output head is the embedding table
     logit_scale: float = 1.0
@@ -420,11 +452,11 @@ class SeqModelConfig:
         layers = []
         for i, L in enumerate(d["layers"]):
             mx, mlp = L["mixer"], L.get("mlp")
-            ff, moe = 0, None
+            ff, moe, ff_limit = 0, None, 0.0
             if mlp is not None:
                 kind = mlp.get("kind", "moe" if "router" in mlp else "dense")
                 if kind == "dense":
-                    ff = int(mlp["ff"])
+                    ff, ff_limit = int(mlp["ff"]), float(mlp.get("limit") or 0.0)
                 elif kind == "moe":
                     r, sh, gr = mlp["router"], mlp.get("shared"), mlp["router"].get("groups")
                     moe = MoeConfig(experts=int(r["experts"]), top=int(r["top"]), ff=int(mlp["expert"]["ff"]),
@@ -433,7 +465,7 @@ class SeqModelConfig:
                                     groups=int(gr["count"]) if gr else 0, keep=int(gr["keep"]) if gr else 0,
                                     act=fam.get("expert", "relu2"), limit=float(mlp["expert"].get("limit", 0.0)),
                                     group_top=int(fam.get("group_top", 1)), correction=bool(fam.get("correction", True)),
-                                    shared_gate=bool(fam.get("shared_gate", True)))
+                                    shared_gate=bool(fam.get("shared_gate", True)), router_bias=bool(fam.get("router_bias", False)))
                 else:
                     raise NotImplementedError(f"layer {i}: feed-forward kind {kind!r} is not supported")
             share = L.get("weights_of")
@@ -448,16 +480,18 @@ class SeqModelConfig:
                         break
                     seen.add(share)
                     share = int(nxt)
-            if L["type"] == "attention":
-                if "attention" not in fam:
-                    raise NotImplementedError(f"layer {i}: {arch} has no mixer of type 'attention'")
+            if L["type"] in ATTENTION_TYPES:
+                if L["type"] not in fam:
+                    raise NotImplementedError(f"layer {i}: {arch} has no mixer of type {L['type']!r}")
                 rot = RotaryConfig.from_json(mx["rot"]) if mx.get("rot") else RotaryConfig(0, 10000.0)
-                mask = mx.get("mask") or {}
+                mask, qt, src = mx.get("mask") or {}, mx.get("q_temp") or {}, mx.get("kv_from")
                 layers.append(SeqLayerConfig("attention", ff=ff, moe=moe, weights_of=-1 if share is None else share, attn=MaskedAttnConfig(
                     heads=int(mx["heads"]), kv_heads=int(mx.get("kv_heads", mx["heads"])), dim=int(mx["dim"]),
                     vdim=int(mx.get("vdim", mx["dim"])), window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0),
                     softcap=float(mx.get("softcap") or 0.0), diff=float(mx.get("diff", 0.0)),
-                    scale=float(mx.get("scale", float(mx["dim"]) ** -0.5)), rot=rot, v_mix=bool(mx.get("v_mix", False)), **fam["attention"])))
+                    scale=float(mx.get("scale", float(mx["dim"]) ** -0.5)), rot=rot, v_mix=bool(mx.get("v_mix", False)),
+                    rel_max=float(mx.get("bias_max") or 0.0), rel_rows=int(mx.get("bias_rows") or 0), temp_coef=float(qt.get("coef", 0.0)),
+                    temp_every=int(qt.get("every", 0)), kv_from=-1 if src is None else int(src), kind=L["type"], **fam[L["type"]])))
             elif L["type"] == "channel_delta":
                 layers.append(SeqLayerConfig("channel_delta", ff=ff, moe=moe, delta=DeltaConfig(
                     heads=int(mx["heads"]), kv_heads=int(mx.get("kv_heads", mx["heads"])), dim=int(mx["dim"]),
@@ -481,7 +515,8 @@ class SeqModelConfig:
                     heads=int(mx["heads"]), dim=int(mx["dim"]), rot_dim=int(mx["rot_dim"]), vdim=int(mx.get("vdim", mx["dim"])),
                     kv_rank=int(mx["kv_rank"]), scale=float(mx["scale"]), rot=RotaryConfig.from_json(mx["rot"], int(mx["rot_dim"])),
                     kv_from=-1 if src is None else int(src), q_rank=int(mx.get("q_rank", 0)) if lf.get("q_latent") else 0,
-                    window=int((mx.get("mask") or {}).get("size", 0)), gate=lf.get("gate", True), sink=lf.get("sink", True))))
+                    window=int((mx.get("mask") or {}).get("size", 0)), gate=lf.get("gate", True), sink=lf.get("sink", True),
+                    gate_channel=lf.get("gate_channel", False), rot_pairs=lf.get("rot_pairs", False))))
             elif L["type"] == "mamba2":
                 layers.append(SeqLayerConfig("mamba2", ssd=SsdMixerConfig(
                     heads=int(mx["heads"]), vdim=int(mx["vdim"]), state=int(mx["state"]), groups=int(mx.get("groups", 1)),
@@ -496,6 +531,7 @@ class SeqModelConfig:
                 layers.append(SeqLayerConfig("parallel", left=left, right=right, ff=ff, moe=moe))
             else:
                 raise NotImplementedError(f"layer {i}: mixer type {L['type']!r} is not supported")
+            layers[-1].ff_limit = ff_limit
         return SeqModelConfig(
             architecture=arch, vocab=int(d["vocab"]), width=int(d["width"]), layers=layers,
             eps=float((d.get("norm") or {}).get("eps", 1e-5)), alpha=float(d.get("postln_alpha", 1.0)),
@@ -503,7 +539,8 @@ class SeqModelConfig:
             eos_token_id=int(d.get("eos_token_id", -1)), block=fam["block"], streams=int(d.get("streams", 1)),
             norm_offset=fam["norm_offset"], positions=fam["positions"], norm=fam.get("norm", "rms"), dense=fam.get("dense", "glu"),
             logit_scale=float(d.get("logit_scale", 1.0)), canon_taps=int((d.get("canon") or {}).get("taps", 0)),
-            norm_scalar=bool(fam.get("norm_scalar", False)), dense_act=fam.get("dense_act", "gelu_tanh"), tied_head=bool(fam.get("tied_head", False)))
+            norm_scalar=bool(fam.get("norm_scalar", False)), dense_act=fam.get("dense_act", "gelu_tanh"), tied_head=bool(fam.get("tied_head", False)),
+            layer_scale=bool(fam.get("layer_scale", False)))
 
     def to_json(self) -> dict:
         """The inverse of from_json (used to write synthetic checkpoints)."""
@@ -530,8 +567,16 @@ class SeqModelConfig:
             elif L.type == "attention":
                 a = L.attn
                 mx = dict(heads=a.heads, kv_heads=a.kv_heads, dim=a.dim, vdim=a.vdim, scale=a.scale, rot=a.rot.to_json())
-                if not a.rot.dims and a.maps > 1:
+                if not a.rot.dims and (a.maps > 1 or a.rel_max):
                     del mx["rot"]
+                if a.rel_max:
+                    mx["bias_max"] = a.rel_max
+                if a.rel_rows:
+                    mx["bias_rows"] = a.rel_rows
+                if a.temp_every:
+                    mx["q_temp"] = dict(coef=a.temp_coef, every=a.temp_every)
+                if a.kv_from >= 0:
+                    mx["kv_from"] = a.kv_from
                 if a.window:
                     mx["mask"] = dict(size=a.window)
                     if a.keep_first:
@@ -554,6 +599,8 @@ class SeqModelConfig:
                 mx = dict(left=dict(heads=l.heads, kv_heads=l.kv_heads, dim=l.dim, vdim=l.vdim, mask=dict(size=l.chunk), scale=l.scale),
                           right=dict(heads=r.heads, dim=r.dim, vdim=r.vdim, tau=r.tau))
             mlp = dict(ff=L.ff, kind="dense") if L.ff else None
+            if L.ff and L.ff_limit:
+                mlp["limit"] = L.ff_limit
             if L.moe:
                 e = L.moe
                 mlp = dict(kind="moe", expert=dict(ff=e.ff), router=dict(experts=e.experts, top=e.top, scale=e.scale))
@@ -561,13 +608,13 @@ class SeqModelConfig:
                     mlp["shared"] = dict(ff=e.shared_ff)
                 if e.act == "clamp_glu":
                     mlp["expert"]["limit"] = e.limit
-                if e.act != "relu2":
+                if e.act != "relu2" or e.router == "topk_softmax":
                     del mlp["router"]["scale"]
                 if e.identity:
                     mlp["router"]["identity"] = e.identity
                 if e.groups:
                     mlp["router"]["groups"] = dict(count=e.groups, keep=e.keep)
-            out.append(dict(type=L.type, mixer=mx, mlp=mlp))
+            out.append(dict(type=L.attn.kind if L.type == "attention" else L.type, mixer=mx, mlp=mlp))
             if L.weights_of >= 0:
                 out[-1]["weights_of"] = L.weights_of
         if self.block == "sandwich":
@@ -603,8 +650,10 @@ class SeqModelConfig:
                 raise ValueError(f"layer {i}: identity experts and a shared expert do not combine")
             if L.weights_of >= 0 and self.block != "parallel":
                 raise ValueError(f"layer {i}: shared layer weights are served in parallel blocks only")
-            if L.moe and L.moe.router == "topk_softmax" and (L.moe.identity or L.moe.groups or L.moe.shared_ff):
-                raise ValueError(f"layer {i}: weights over the chosen logits combine with neither identity experts, groups nor a shared expert")
+            if L.moe and L.moe.router == "topk_softmax" and (L.moe.identity or L.moe.groups):
+                raise ValueError(f"layer {i}: weights over the chosen logits combine with neither identity experts nor groups")
+            if L.ff and self.dense == "clamp_glu" and not L.ff_limit > 0:
+                raise ValueError(f"layer {i}: a clamped gated feed-forward needs its limit")
             if L.type == "channel_delta":
                 t = L.delta
                 if t.heads < 1 or t.kv_heads < 1 or t.heads % t.kv_heads or not 1 <= t.dim <= 512 or t.vdim < 1 or not 1 <= t.conv <= 8:
@@ -612,8 +661,15 @@ class SeqModelConfig:
                 continue
             if L.type == "attention":
                 a = L.attn
-                if self.block not in ("parallel", "branchnorm", "sandwich"):
-                    raise ValueError(f"layer {i}: the attention mixer is served in parallel blocks and in blocks normed on the sublayer's output")
+                if self.block == "prenorm_hc":
+                    raise ValueError(f"layer {i}: the attention mixer is not served in blocks on several streams")
+                if a.rel_max < 0 or a.temp_every < 0 or a.rel_rows < 0:
+                    raise ValueError(f"layer {i}: unsupported distance bias or query temperature {a}")
+                if a.kv_from >= 0:
+                    o = self.layers[a.kv_from] if a.kv_from < i else None
+                    if o is None or o.type != "attention" or o.attn.kv_from >= 0 or a.maps > 1 or a.v_mix or a.value_keys or \
+                            (o.attn.kv_heads, o.attn.dim, o.attn.vdim, o.attn.maps) != (a.kv_heads, a.dim, a.vdim, a.maps):
+                        raise ValueError(f"layer {i}: kv_from must name an earlier attention layer with its own cache and the same geometry")
                 if a.maps not in (1, 2) or a.keep_first < 0 or a.softcap < 0 or a.vdim < 1:
                     raise ValueError(f"layer {i}: unsupported attention options {a}")
                 if a.v_mix:

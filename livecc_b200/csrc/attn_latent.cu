@@ -30,7 +30,7 @@ __global__ void __launch_bounds__(256) latent_kv_append_kernel(const T* __restri
                                                                const float* __restrict__ inv_freq, float mag,
                                                                float* __restrict__ q_out, T* __restrict__ k_pages,
                                                                const int* __restrict__ page_table, int page_size, int H, int D,
-                                                               int DR, int R, SeqPos pos, const T* __restrict__ qsrc, int ld_q) {
+                                                               int DR, int R, SeqPos pos, const T* __restrict__ qsrc, int ld_q, bool pairs) {
     if (seq_done(pos)) return;
     __shared__ float red[32];
     const int t = blockIdx.x;
@@ -38,15 +38,18 @@ __global__ void __launch_bounds__(256) latent_kv_append_kernel(const T* __restri
     const float p = (float)pi;
     const T* row = proj + (size_t)t * ld;
     const int half = DR / 2, QH = D + DR, nq = H * QH, KD = R + DR;
+    // channel r of the rotated part: its pair's angle, its partner, and whether it is the pair's first member
+    auto turned = [&](const T* x, int r) {
+        const bool first = pairs ? !(r & 1) : r < half;
+        const float ang = p * inv_freq[pairs ? r >> 1 : (first ? r : r - half)];
+        const float c = cosf(ang) * mag, s = sinf(ang) * mag;
+        const float v = ldf(x + r), other = ldf(x + (pairs ? r ^ 1 : (first ? r + half : r - half)));
+        return first ? v * c - other * s : v * c + other * s;
+    };
     // rotated query part of every head -> q_out[t, h, R + j]
     for (int i = threadIdx.x + blockIdx.y * blockDim.x; i < H * DR; i += blockDim.x * gridDim.y) {
         const int h = i / DR, r = i % DR;
-        const int j = r < half ? r : r - half;
-        const float ang = p * inv_freq[j];
-        const float c = cosf(ang) * mag, s = sinf(ang) * mag;
-        const T* qr = (qsrc ? qsrc + (size_t)t * ld_q : row) + (size_t)h * QH + D;
-        const float v = ldf(qr + r), other = ldf(qr + (r < half ? r + half : r - half));
-        q_out[((size_t)t * H + h) * KD + R + r] = r < half ? v * c - other * s : v * c + other * s;
+        q_out[((size_t)t * H + h) * KD + R + r] = turned((qsrc ? qsrc + (size_t)t * ld_q : row) + (size_t)h * QH + D, r);
     }
     if (!has_kv || blockIdx.y != 0) return;
     const T* lat = qsrc ? row : row + nq;      // queries of their own: the row starts with the latent
@@ -56,30 +59,24 @@ __global__ void __launch_bounds__(256) latent_kv_append_kernel(const T* __restri
     const float rn = 1.f / sqrtf(ss / (float)R + eps);
     T* dst = k_pages + ((size_t)page_table[pi / page_size] * page_size + pi % page_size) * KD;
     for (int i = threadIdx.x; i < R; i += blockDim.x) stf(dst + i, ldf(lat + i) * rn * norm_w[i]);
-    for (int r = threadIdx.x; r < DR; r += blockDim.x) {
-        const int j = r < half ? r : r - half;
-        const float ang = p * inv_freq[j];
-        const float c = cosf(ang) * mag, s = sinf(ang) * mag;
-        const float v = ldf(lat + R + r), other = ldf(lat + R + (r < half ? r + half : r - half));
-        stf(dst + R + r, r < half ? v * c - other * s : v * c + other * s);
-    }
+    for (int r = threadIdx.x; r < DR; r += blockDim.x) stf(dst + R + r, turned(lat + R, r));
 }
 
 }  // namespace
 
 int latent_kv_append(int dt, const void* proj, int ld, int has_kv, const float* norm_w, float eps, const float* inv_freq,
                      float mag, float* q_out, void* k_pages, const int* page_table, int page_size, int S, int H, int D,
-                     int DR, int R, SeqPos pos, cudaStream_t s, const void* q, int ld_q) {
+                     int DR, int R, SeqPos pos, cudaStream_t s, const void* q, int ld_q, bool rot_pairs) {
     if (!proj || !inv_freq || !q_out || S < 1 || H < 1 || D < 0 || DR < 2 || (DR & 1) || R < 1) return -2;
     if (has_kv && (!norm_w || !k_pages || !page_table || page_size < 1)) return -2;
     count_launch();
     const dim3 S_grid(S, S < 32 ? 4 : 1);
     if (dt == DT_F32)
         latent_kv_append_kernel<float><<<S_grid, 256, 0, s>>>((const float*)proj, ld, has_kv, norm_w, eps, inv_freq, mag, q_out,
-                                                         (float*)k_pages, page_table, page_size, H, D, DR, R, pos, (const float*)q, ld_q);
+                                                         (float*)k_pages, page_table, page_size, H, D, DR, R, pos, (const float*)q, ld_q, rot_pairs);
     else
         latent_kv_append_kernel<bf16><<<S_grid, 256, 0, s>>>((const bf16*)proj, ld, has_kv, norm_w, eps, inv_freq, mag, q_out,
-                                                        (bf16*)k_pages, page_table, page_size, H, D, DR, R, pos, (const bf16*)q, ld_q);
+                                                        (bf16*)k_pages, page_table, page_size, H, D, DR, R, pos, (const bf16*)q, ld_q, rot_pairs);
     return cudaGetLastError() == cudaSuccess ? 0 : -100;
 }
 

@@ -3,7 +3,8 @@
 //   * attention of new rows over the keys of their own chunk (chunks counted from position 0 of the sequence) with a
 //     softmax sink: p_j = exp(s_j) / (exp(sink_h) + sum_j exp(s_j)) (sink_h = 0 unless given), and a per-head sigmoid output gate.
 // Options (AttnOpts): a sliding window instead of / inside the chunks that may keep the first positions, no sink (ordinary softmax),
-// one gate per output channel, soft-capped scores, two maps per head whose difference is the output (differential attention).
+// one gate per output channel, soft-capped scores, a bias per head and distance, two maps per head whose difference is the output
+// (differential attention).
 // Scores, weights and the accumulation are fp32; K and V pages hold the model's storage type.
 #include <math.h>
 #include <stdlib.h>
@@ -42,6 +43,8 @@ __device__ __forceinline__ float soft_cap_fast(float s, float cap, float inv_cap
     const float e = __expf(2.f * fminf(s * inv_cap, 40.f));
     return cap - __fdividef(2.f * cap, 1.f + e);
 }
+// A head's bias by distance: row h of the table [heads][len]; distances from len - 1 on share its last entry (AttnOpts::bias)
+__device__ __forceinline__ float bias_at(const float* row, int len, int dist) { return __ldg(row + min(dist, len - 1)); }
 // With a window that keeps the first `keep` positions, a row whose window starts at `lo` sees [0, keep) and [lo, p]. The key tiles of
 // a group of rows whose first window starts at `kbeg` are walked from `k_start` on; a step from a tile of the kept positions skips
 // what lies between them and kbeg.
@@ -88,7 +91,10 @@ __global__ void __launch_bounds__(256) qk_headnorm_rope_append_kernel(const T* _
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
     const int page = page_table[p / page_size], slot = p % page_size;
     const int half = rot_dims >> 1;
-    for (int hd = blockIdx.y * nwarps + warp; hd < Hq + G; hd += gridDim.y * nwarps) {
+    // a temperature on the queries that grows with the position, in steps of `every` positions
+    const float q_temp = ao.temp_every > 0 ? fmaf(ao.temp_coef, logf((float)((p + 1) / ao.temp_every + 1)), 1.f) : 1.f;
+    const int n_heads = ao.q_only ? Hq : Hq + G;
+    for (int hd = blockIdx.y * nwarps + warp; hd < n_heads; hd += gridDim.y * nwarps) {
         const bool is_q = hd < Hq;
         const T* x = row + (size_t)hd * D;                 // k heads follow the q heads in the row
         const float* w = is_q ? qn_w : kn_w;
@@ -105,7 +111,7 @@ __global__ void __launch_bounds__(256) qk_headnorm_rope_append_kernel(const T* _
             }
             for (int j = lane + 32 * kKeep; j < np; j += 32) { const float2 v = ld2(x + 2 * j); ss = fmaf(v.x, v.x, fmaf(v.y, v.y, ss)); }
             ss = warp_sum(ss);
-            const float rn = ((w || ao.unit_norm) ? 1.f / sqrtf(ss / (float)D + eps) : 1.f) * ((is_q && ao.q_head_scale) ? ao.q_head_scale[hd] : 1.f);
+            const float rn = ((w || ao.unit_norm) ? 1.f / sqrtf(ss / (float)D + eps) : 1.f) * ((is_q && ao.q_head_scale) ? ao.q_head_scale[hd] : 1.f) * (is_q ? q_temp : 1.f);
             float* qo = q_out + ((size_t)t * Hq + hd) * D;
             T* ko = k_pages + (((size_t)page * G + (hd - Hq)) * page_size + slot) * D;
             auto emit = [&](int j, const float2 v) {
@@ -127,7 +133,7 @@ __global__ void __launch_bounds__(256) qk_headnorm_rope_append_kernel(const T* _
         }
         for (int c = lane; c < D; c += 32) { const float v = ldf(x + c); ss = fmaf(v, v, ss); }
         ss = warp_sum(ss);
-        const float rn = ((w || ao.unit_norm) ? 1.f / sqrtf(ss / (float)D + eps) : 1.f) * ((is_q && ao.q_head_scale) ? ao.q_head_scale[hd] : 1.f);
+        const float rn = ((w || ao.unit_norm) ? 1.f / sqrtf(ss / (float)D + eps) : 1.f) * ((is_q && ao.q_head_scale) ? ao.q_head_scale[hd] : 1.f) * (is_q ? q_temp : 1.f);
         for (int c = lane; c < D; c += 32) {
             float v = ldf(x + c) * rn * (w ? w[c] : 1.f);
             if (c < rot_dims) {
@@ -146,7 +152,7 @@ __global__ void __launch_bounds__(256) qk_headnorm_rope_append_kernel(const T* _
             else stf(k_pages + (((size_t)page * G + (hd - Hq)) * page_size + slot) * D + c, v);
         }
     }
-    const int nv = G * DV;
+    const int nv = ao.q_only ? 0 : G * DV;
     for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < nv; i += gridDim.y * blockDim.x) {
         const int g = i / DV, d = i % DV;
         T* dst = v_pages + (((size_t)page * G + g) * page_size + slot) * DV + d;
@@ -206,6 +212,7 @@ __global__ void __launch_bounds__(128) attn_chunk_sink_kernel(const float* __res
     const int start = first_key(p, chunk, opt.window);
     const int nkeep = min(opt.keep_first, start), nkeys = p - start + 1 + nkeep;   // key jk: the kept positions, then the window's
     const int ld_k = D * opt.maps, koff = (h % opt.maps) * D;
+    const float* brow = opt.bias ? opt.bias + (size_t)(h / opt.maps) * opt.bias_len : nullptr;
     float* sq = sm;           // [D]
     float* sc = sm + D;       // [nkeys]
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
@@ -220,6 +227,7 @@ __global__ void __launch_bounds__(128) attn_chunk_sink_kernel(const float* __res
         for (int d = lane; d < D; d += 32) acc = fmaf(sq[d], ldf(kr + d), acc);
         acc = warp_sum(acc) * scale;
         if (opt.softcap > 0.f) acc = soft_cap(acc, opt.softcap, 1.f / opt.softcap);
+        if (brow) acc += bias_at(brow, opt.bias_len, p - pj);
         if (lane == 0) sc[jk] = acc;
         mx = fmaxf(mx, acc);
     }
@@ -291,6 +299,7 @@ __global__ void __launch_bounds__(128) attn_split_kernel(const float* __restrict
     __shared__ float red[32];
     __shared__ float redm[4];
     __shared__ int row_of[kSplitKeys];     // a key's row in the page pool: (page * G + g) * page_size + slot
+    __shared__ float bias_of[kSplitKeys];  // and what its distance adds to its score
     __shared__ int last_flag;
     float* sq = sm;            // [D]
     float* sc = sm + D;        // [kSplitKeys]
@@ -300,6 +309,7 @@ __global__ void __launch_bounds__(128) attn_split_kernel(const float* __restrict
     const int kfirst = first_key(npos - 1, 0, opt.window), nkeep = min(opt.keep_first, kfirst), nkeys = npos - kfirst + nkeep;
     const int ld_k = D * opt.maps, koff = (h % opt.maps) * D;
     const float inv_cap = opt.softcap > 0.f ? 1.f / opt.softcap : 0.f;
+    const float* brow = opt.bias ? opt.bias + (size_t)(h / opt.maps) * opt.bias_len : nullptr;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     for (int i = threadIdx.x; i < D; i += blockDim.x) sq[i] = q[((size_t)t * Hq + h) * D + i] * scale;
     float m = -INFINITY, l = 0.f;
@@ -314,6 +324,7 @@ __global__ void __launch_bounds__(128) attn_split_kernel(const float* __restrict
         for (int j = threadIdx.x; j < nk; j += blockDim.x) {
             const int pj = k0 + j < nkeep ? k0 + j : kfirst + k0 + j - nkeep;
             row_of[j] = (int)(((size_t)page_table[pj / page_size] * G + g) * page_size + pj % page_size);
+            if (brow) bias_of[j] = bias_at(brow, opt.bias_len, npos - 1 - pj);
         }
         __syncthreads();
         float mx = -INFINITY;
@@ -351,6 +362,7 @@ __global__ void __launch_bounds__(128) attn_split_kernel(const float* __restrict
                 float v = warp_sum(acc[j]);
                 if (opt.softcap > 0.f) v = soft_cap(v, opt.softcap, inv_cap);
                 if (j0 + j < nk) {
+                    if (brow) v += bias_of[j0 + j];
                     if (lane == 0) sc[j0 + j] = v;
                     mx = fmaxf(mx, v);
                 }
@@ -541,6 +553,7 @@ __global__ void __launch_bounds__(256) attn_chunk_sink_tiled_kernel(const float*
     const int keep = min(opt.keep_first, kbeg), k_start = keep > 0 ? 0 : kbeg;
     const int ld_k = D * opt.maps, koff = (h % opt.maps) * D;
     const float inv_cap = opt.softcap > 0.f ? 1.f / opt.softcap : 0.f;
+    const float* brow = opt.bias ? opt.bias + (size_t)(h / opt.maps) * opt.bias_len : nullptr;
     const int tm = (threadIdx.x / 16) * 4, tn = (threadIdx.x % 16) * 4;
     const int lr = threadIdx.x / 16, lc = threadIdx.x % 16;              // staging: 16 threads walk a row
     int p_row[4], lo_row[4];
@@ -621,7 +634,8 @@ __global__ void __launch_bounds__(256) attn_chunk_sink_tiled_kernel(const float*
                 const int pj = k0 + tn + j;
                 const bool ok = pj <= p_row[i] && (pj >= lo_row[i] || pj < opt.keep_first) && tm + i < rows;
                 const float v = sc[i][j] * scale;
-                sc[i][j] = ok ? (opt.softcap > 0.f ? soft_cap(v, opt.softcap, inv_cap) : v) : -INFINITY;
+                sc[i][j] = ok ? (opt.softcap > 0.f ? soft_cap(v, opt.softcap, inv_cap) : v) + (brow ? bias_at(brow, opt.bias_len, p_row[i] - pj) : 0.f)
+                              : -INFINITY;
                 mx = fmaxf(mx, sc[i][j]);
             }
 #pragma unroll
@@ -715,7 +729,9 @@ __device__ __forceinline__ void stage_bf16_rows(bf16* dst, int n_rows, int ld_ds
 // MAPS = 2 (differential attention; KH = 2): the two groups of warps take the two maps of one head over the SAME key tiles, so a tile's
 // V rows are staged once for both; at the end the second group hands its normalised output to the first, which writes the normed
 // difference. D is a map's width; key rows hold both maps.
-// EXT: soft-capped scores, kept first positions, key rows of two maps, fp32 output of one map (compiled out of the plain form).
+// EXT: soft-capped scores, distance biases, kept first positions, key rows of two maps, fp32 output of one map (compiled out of the
+// plain form). A 64 x 64 tile of scores meets 127 distances: their biases are staged in shared memory beside the tile's keys, and a
+// tile whose distances all lie past the table adds its last entry.
 template <bool VEC8, int KH, int NV, int NBUF = 2, int MAPS = 1, bool EXT = false>
 __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 : 0) attn_chunk_sink_mma_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pages,
                                                                   const bf16* __restrict__ v_pages, const int* __restrict__ page_table,
@@ -744,6 +760,9 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 :
     // a CTA of one map works on head h = head * opt.maps + map (its K columns start at map * D), a CTA of both maps on head h
     const int ld_k = EXT ? D * opt.maps : D, koff = EXT && MAPS == 1 ? (h % opt.maps) * D : 0;
     const float inv_cap = EXT && opt.softcap > 0.f ? 1.f / opt.softcap : 0.f;
+    __shared__ float sbias[EXT ? 2 * KH * 128 : 1];     // [step parity][group of warps][distance]
+    const float* brow = EXT && opt.bias ? opt.bias + (size_t)(MAPS == 2 ? h : h / opt.maps) * opt.bias_len : nullptr;
+    const float far_bias = brow ? brow[opt.bias_len - 1] : 0.f;
     const int dvv = min(MVW, DV - c0), DVp = (dvv + 15) / 16 * 16;
     const int warp = (threadIdx.x >> 5) & 3, kh = threadIdx.x >> 7, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
     // queries: fp32 -> bf16, zero padding
@@ -800,6 +819,11 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 :
         const int k0 = MAPS == 2 ? kc : kc + kh * MK;   // this group of warps' tile of the step
         const bf16* sK = sK0 + ((size_t)buf * KR + kh * MK) * LQ;
         const bf16* sV = sV0 + ((size_t)buf * KT + (MAPS == 2 ? 0 : kh * MK)) * MLV;
+        // entry u: the bias of distance pf - k0 + u - (MK - 1) (row r and key c meet at u = r - c + MK - 1). The other parity's entries
+        // may still be read; this parity's last readers are behind the barrier of the step before.
+        const bool near = EXT && brow && pf - (k0 + MK - 1) < opt.bias_len - 1;
+        float* sb = sbias + (EXT ? ((it & 1) * KH + kh) * 128 : 0);
+        if (near) sb[threadIdx.x & 127] = bias_at(brow, opt.bias_len, max(pf - k0 + (int)(threadIdx.x & 127) - (MK - 1), 0));
         if (VEC8 && NBUF == 1) {
             __syncthreads();       // every thread is done with the previous tile (and Q is staged)
             issue(kc, 0);
@@ -855,6 +879,7 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 :
                 for (int e = 0; e < 2; ++e) {
                     float v = sc[j][2 * i + e] * scale;
                     if (EXT && opt.softcap > 0.f) v = soft_cap_fast(v, opt.softcap, inv_cap);
+                    if (EXT && brow) v += near ? sb[r_lo + 8 * i + MK - 1 - (j * 8 + 2 * tq + e)] : far_bias;
                     if (!full) {
                         const int pj = k0 + j * 8 + 2 * tq + e;
                         const bool ok = pj <= p_row[i] && (pj >= lo_row[i] || (EXT && pj < keep_first)) && r_lo + 8 * i < rows;
@@ -1013,8 +1038,8 @@ __global__ void __launch_bounds__(128 * KH, (VEC8 && NBUF == 1 && NV == 1) ? 2 :
 int launch_attn_mma(const float* q, const void* k_pages, const void* v_pages, const int* page_table, int page_size,
                     const void* gate, int ld_gate, void* out, int ld_out, int S, int Hq, int G, int D, int DV, int chunk,
                     float scale, SeqPos pos, cudaStream_t s, const float* sink, int ld_v, AttnOpts opt) {
-    static SmemAttrOnce once82, once82s, once81, once1, once81w, once1w, once81x, once1x, once81wx, once1wx;
-    const bool ext = opt.softcap > 0.f || opt.keep_first > 0 || opt.maps > 1;
+    static SmemAttrOnce once82, once82s, once81, once1, once81w, once1w, once81x, once1x, once81wx, once1wx, once82x;
+    const bool ext = opt.softcap > 0.f || opt.keep_first > 0 || opt.maps > 1 || opt.bias;
     // two groups of warps: one K/V buffer and two CTAs per SM (default), or two buffers and one CTA (LIVECC_B200_SEQ_ATTN_NBUF=2)
     static const int nbuf2 = [] { const char* e = getenv("LIVECC_B200_SEQ_ATTN_NBUF"); return e ? atoi(e) : 1; }();
     const int Dp = (D + 15) / 16 * 16;
@@ -1024,8 +1049,8 @@ int launch_attn_mma(const float* q, const void* k_pages, const void* v_pages, co
     // merge (68 floats per thread of a group, 34 KB) lies over the K and V buffers, whose V part alone is 68 KB
     // values wider than 128 channels: two output tiles per CTA against one pass over the scores (one group of warps)
     const bool wide = DV > 128;
-    const bool two = vec8 && Dp <= 128 && !wide && !ext;
-    const int nbuf = vec8 ? ((two && nbuf2 == 1) ? 1 : 2) : 1, kh = two ? 2 : 1, MVW = wide ? 256 : 128, MLV = MVW + 8;
+    const bool two = vec8 && Dp <= 128 && !wide && (!ext || opt.maps == 1);
+    const int nbuf = vec8 ? ((two && (nbuf2 == 1 || ext)) ? 1 : 2) : 1, kh = two ? 2 : 1, MVW = wide ? 256 : 128, MLV = MVW + 8;
     auto bytes = [&](int dp) { return ((size_t)MQ * (dp + 8) + (size_t)nbuf * kh * MK * (dp + 8 + MLV)) * sizeof(bf16); };
     const size_t smem = bytes(Dp), smem_max = bytes(two ? 128 : kAttnMmaMaxDim);
     dim3 grid(Hq, (S + MQ - 1) / MQ, (DV + MVW - 1) / MVW);
@@ -1039,6 +1064,7 @@ int launch_attn_mma(const float* q, const void* k_pages, const void* v_pages, co
     } while (0)
     if (ext && wide && vec8) LCC_ATTN_MMA(once81wx, true, 1, 2, 2, 1, true);
     else if (ext && wide) LCC_ATTN_MMA(once1wx, false, 1, 2, 2, 1, true);
+    else if (ext && two) LCC_ATTN_MMA(once82x, true, 2, 1, 1, 1, true);
     else if (ext && vec8) LCC_ATTN_MMA(once81x, true, 1, 1, 2, 1, true);
     else if (ext) LCC_ATTN_MMA(once1x, false, 1, 1, 2, 1, true);
     else if (two && nbuf == 1) LCC_ATTN_MMA(once82s, true, 2, 1, 1);
@@ -1137,14 +1163,15 @@ int qk_headnorm_rope_append(int dt, const void* proj, int ld, int v_col, const f
                             void* v_pages, const int* page_table, int page_size, int S, int Hq, int G, int D, int DV, SeqPos pos,
                             cudaStream_t s, const AppendOpts* opt) {
     if (!proj || !q_out || !k_pages || !v_pages || !page_table || S < 1 || Hq < 1 || G < 1 || D < 1 || DV < 1 || page_size < 1 ||
-        rot_dims < 0 || (rot_dims & 1) || rot_dims > D || (rot_dims > 0 && !inv_freq) || v_col < 0 || v_col + G * DV > ld)
+        rot_dims < 0 || (rot_dims & 1) || rot_dims > D || (rot_dims > 0 && !inv_freq) || v_col < 0)
         return -2;
     const AppendOpts ao = opt ? *opt : AppendOpts{false, nullptr, nullptr, 0, 0.f, nullptr, 0};
+    if (ao.temp_every < 0 || (ao.q_only ? (Hq * D > ld || ao.v_mix || ao.v_keep) : v_col + G * DV > ld)) return -2;
     if ((ao.v_mix && ao.ld_mix < G * DV) || (ao.v_keep && ao.ld_keep < G * DV)) return -2;
     count_launch();
     // many rows: 8 warps walk a row's heads; few rows: 4-warp CTAs, one head per warp, so that a decode step fills more SMs
     const int threads = S >= 64 ? 256 : 128;
-    const dim3 grid(S, S >= 64 ? 1 : (Hq + G + 3) / 4);
+    const dim3 grid(S, S >= 64 ? 1 : (Hq + (ao.q_only ? 0 : G) + 3) / 4);
     const size_t es = dt == DT_F32 ? 4 : 2;
     const bool pairs = (rot_pairs || rot_dims == 0) && (D % 2) == 0 && (ld % 2) == 0 && ((uintptr_t)proj % (2 * es)) == 0 &&
                        ((uintptr_t)k_pages % (2 * es)) == 0 && ((uintptr_t)q_out % 8) == 0;
@@ -1168,6 +1195,7 @@ int attn_masked(int dt, const float* q, const void* k_pages, const void* v_pages
     if (ld_v < DV) return -2;
     if (opt.maps != 1 && (opt.maps != 2 || gate || !opt.raw)) return -2;
     if (opt.maps == 1 && opt.raw) return -2;
+    if (opt.bias && opt.bias_len < 1) return -2;
     const int window = opt.window > 0 ? opt.window : 0;
     if (opt.keep_first < 0 || (opt.keep_first > 0 && chunk > 0)) return -2;
     const int keep = window ? opt.keep_first : 0;      // (without a window every position stays anyway)

@@ -22,6 +22,8 @@ enum GemmEpilogue {
                              // C[:, j] = bf16(g * sigmoid(alpha g) * (u + up_bias)) in fp32 on the accumulators; limit = epi_param,
                              // alpha = epi_alpha, up_bias = epi_up_bias (1, 0 and an infinite limit: silu(gate) * up)
     EPI_GELU_ERF = 11,       // C = bf16(gelu_erf(acc)), the activation in fp32 on the accumulator
+    EPI_SIGMOID_GATE = 12,   // C = bf16(acc * sigmoid(residual)): the residual slot carries gate logits (batched: product z reads its columns
+                             // z * c_col_stride .. , as it writes C)
 };
 
 struct GemmArgs {

@@ -148,6 +148,16 @@ __device__ __forceinline__ void epilogue_chunk(const uint32_t (&v)[32], bf16* C,
 #pragma unroll
                     for (int j = 0; j < 8; ++j) { x[j] = fmaxf(x[j], 0.f); x[j] *= x[j]; }
                 }
+                if (EPI == EPI_SIGMOID_GATE) {
+                    const uint4 gg = *reinterpret_cast<const uint4*>(residual + (size_t)row * ldr + col);
+                    const uint32_t gw[4] = {gg.x, gg.y, gg.z, gg.w};
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        const float2 f = unpack_bf16x2(gw[j]);
+                        x[2 * j] = __fdividef(x[2 * j], 1.f + __expf(-f.x));
+                        x[2 * j + 1] = __fdividef(x[2 * j + 1], 1.f + __expf(-f.y));
+                    }
+                }
                 if (EPI == EPI_GELU_ERF) {
 #pragma unroll
                     for (int j = 0; j < 8; ++j) x[j] = 0.5f * x[j] * (1.f + erff(x[j] * 0.7071067811865476f));
@@ -336,7 +346,8 @@ gemm_bf16_tn_kernel(const __grid_constant__ CUtensorMap tmap_a,
                 // batched: entry z's columns start at z * c_col_stride (floats when the output is fp32)
                 bf16* Cz = (EPI == EPI_PARTIAL_F32) ? reinterpret_cast<bf16*>(reinterpret_cast<float*>(C) + (size_t)z * c_col_stride)
                                                     : C + (size_t)z * c_col_stride;
-                epilogue_chunk<EPI>(v, Cz, ldc, M, row, row_ok, col0, tile_end, ks, bias, residual, ldr);
+                epilogue_chunk<EPI>(v, Cz, ldc, M, row, row_ok, col0, tile_end, ks, bias,
+                                    EPI == EPI_SIGMOID_GATE ? residual + (size_t)z * c_col_stride : residual, ldr);
             }
             tc_fence_before();
             __syncwarp();
@@ -646,6 +657,7 @@ static int launch_epi(const GemmArgs& a, int bn, int num_sms, cudaStream_t strea
         case EPI_GELU_TANH: return launch_cfg<EPI_GELU_TANH>(a, bn, num_sms, stream);
         case EPI_GELU_ERF: return launch_cfg<EPI_GELU_ERF>(a, bn, num_sms, stream);
         case EPI_CLAMP_GLU: return launch_cfg<EPI_CLAMP_GLU>(a, bn, num_sms, stream);
+        case EPI_SIGMOID_GATE: return launch_cfg<EPI_SIGMOID_GATE>(a, bn, num_sms, stream);
     }
     return -14;
 }
@@ -762,7 +774,8 @@ int gemm_bf16_tn(const GemmArgs& a, int num_sms, cudaStream_t stream) {
     if (a.M <= 0 || a.N <= 0 || a.K <= 0) return -1;
     if ((a.K % 8) || (a.lda % 8) || (a.ldb % 8) || (a.N % 8) || (a.ldc % (a.c_f32 ? 4 : 8))) return -2;
     if ((a.epi == EPI_SWIGLU || a.epi == EPI_CLAMP_GLU) && (a.N % 32)) return -3;
-    if ((a.epi == EPI_RESIDUAL || a.epi == EPI_BIAS_RESIDUAL) && (!a.residual || (a.ldr % 8))) return -4;
+    if ((a.epi == EPI_RESIDUAL || a.epi == EPI_BIAS_RESIDUAL || a.epi == EPI_SIGMOID_GATE) && (!a.residual || (a.ldr % 8))) return -4;
+    if (a.epi == EPI_SIGMOID_GATE && (((uintptr_t)a.residual % 16) || a.tile_group)) return -4;
     if ((a.epi == EPI_BIAS || a.epi == EPI_BIAS_QUICKGELU || a.epi == EPI_BIAS_GELU ||
          a.epi == EPI_BIAS_RESIDUAL) && !a.bias) return -5;
     if (a.tile_group && a.groups < 1) return -1;
@@ -781,7 +794,7 @@ int gemm_bf16_tn(const GemmArgs& a, int num_sms, cudaStream_t stream) {
         block_n = forced > 0 ? forced : choose_bn(a.M, a.N, num_sms);
     }
     // block_n < 0 selects the CTA-pair kernel with tile width -block_n (explicit: tests and tuning)
-    const bool pair = block_n < 0 && plain && a.epi != EPI_RELU2 && a.epi != EPI_GELU_TANH && a.epi != EPI_GELU_ERF && a.epi != EPI_CLAMP_GLU;
+    const bool pair = block_n < 0 && plain && a.epi != EPI_RELU2 && a.epi != EPI_GELU_TANH && a.epi != EPI_GELU_ERF && a.epi != EPI_CLAMP_GLU && a.epi != EPI_SIGMOID_GATE;
     if (block_n < 0) block_n = -block_n;
     if (block_n < 32 || block_n > 256 || (block_n % 16) || ((a.epi == EPI_SWIGLU || a.epi == EPI_CLAMP_GLU) && (block_n % 32))) return -6;
     if (pair) return (block_n % 32) ? -6 : launch_epi2(a, block_n, num_sms, stream);

@@ -31,7 +31,15 @@ struct Grp {
     int glu_il16;
     float glu_limit;
     float glu_alpha, glu_up_bias;   // g * sigmoid(alpha g) * (u + up_bias)
+    const void* gate = nullptr;     // the store multiplies by sigmoid(gate[row, z * gate_stride + column]) (no lists)
+    int ld_gate = 0;
+    int64_t gate_stride = 0;
 };
+template <typename T>
+__device__ __forceinline__ float gated(float v, const Grp& g, int z, int row, int col) {
+    if (!g.gate) return v;
+    return v / (1.f + expf(-ldf((const T*)g.gate + (size_t)row * g.ld_gate + z * g.gate_stride + col)));
+}
 __device__ __forceinline__ float act_of(float v, int act) {
     if (act == ACT_RELU2) { v = fmaxf(v, 0.f); v *= v; }
     else if (act == ACT_GELU_ERF) v = 0.5f * v * (1.f + erff(v * 0.7071067811865476f));
@@ -88,7 +96,7 @@ __global__ void __launch_bounds__(256) linear_tile_kernel(const T* __restrict__ 
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int gn = n0 + tn + j;
-            if (gn < N) stf(C + (size_t)gm * ldc + gn, act_of(acc[i][j] + (bias ? bias[gn] : 0.f), g.act));
+            if (gn < N) stf(C + (size_t)gm * ldc + gn, gated<T>(act_of(acc[i][j] + (bias ? bias[gn] : 0.f), g.act), g, blockIdx.z, gm, gn));
         }
     }
 }
@@ -220,7 +228,7 @@ __global__ void __launch_bounds__(256) linear_rows_kernel(const T* __restrict__ 
         for (int m = 0; m < kRowsMax; ++m) {
             if (m < M) {
                 const float v = warp_sum(acc[r][m]);
-                if (lane == 0 && n < N) stf(C + (size_t)m * ldc + n, act_of(v + (bias ? bias[n] : 0.f), g.act));
+                if (lane == 0 && n < N) stf(C + (size_t)m * ldc + n, gated<T>(act_of(v + (bias ? bias[n] : 0.f), g.act), g, z, mb + m, n));
             }
         }
     }
@@ -295,7 +303,9 @@ int linear_grouped(const GroupedLinear& q, cudaStream_t s) {
     if (q.glu_F > 0 && (q.N != q.glu_F || q.act != ACT_NONE || q.c_f32 || (q.glu_il16 && (q.glu_F % 16)) || q.c_stride != 0 ||
                         (q.groups > 1 && !q.row_off)))
         return -2;
-    const Grp g{q.a_stride, q.w_stride, q.c_stride, q.row_off, q.a_rows, q.act, 0, q.glu_F, q.glu_il16 ? 1 : 0, q.glu_limit, q.glu_alpha, q.glu_up_bias};
+    if (q.gate && (q.row_off || q.glu_F > 0)) return -2;
+    const Grp g{q.a_stride, q.w_stride, q.c_stride, q.row_off, q.a_rows, q.act, 0, q.glu_F, q.glu_il16 ? 1 : 0, q.glu_limit, q.glu_alpha, q.glu_up_bias,
+                q.gate, q.ld_gate, q.gate_stride};
     const int mt = q.row_off ? (q.M_total > 0 ? q.M_total : q.M * q.groups) : 0;
     if (q.dt == DT_F32) return launch_linear<float, float>(q.A, q.lda, q.W, q.ldw, nullptr, q.C, q.ldc, q.M, q.N, q.K, s, q.groups, g, mt, q.glu_tmp, q.ld_tmp);
     if (q.c_f32) return launch_linear<bf16, float>(q.A, q.lda, q.W, q.ldw, nullptr, q.C, q.ldc, q.M, q.N, q.K, s, q.groups, g, mt);

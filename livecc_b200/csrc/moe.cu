@@ -1,6 +1,6 @@
 // Mixture-of-experts routing: a sigmoid or softmax router with a choice-only correction (optionally limited to the best
 // groups of neighbouring experts, optionally with identity experts that own no list), the expert-sorted row lists that the
-// grouped linear kernels walk, and the weighted combine. Router scores, weights and gates are fp32.
+// grouped linear kernels walk. Router scores, weights and gates are fp32.
 #include <math.h>
 
 #include "common.cuh"
@@ -31,13 +31,14 @@ template <typename Emit>
 __device__ __forceinline__ void route_row(const float* __restrict__ z, const float* __restrict__ correction, int E, int top,
                                           const MoeRouterOpts& ro, float* gch, unsigned char* gkeep, Emit emit) {
     const int lane = threadIdx.x & 31;
+    auto logit = [&](int e) { return z[e] + (ro.logit_bias ? ro.logit_bias[e] : 0.f); };
     float sc[kMaxExpertsPerLane], ch[kMaxExpertsPerLane];
     float zmax = -INFINITY, zsum = 0.f;
     if (ro.softmax) {
 #pragma unroll
         for (int i = 0; i < kMaxExpertsPerLane; ++i) {
             const int e = lane + 32 * i;
-            sc[i] = e < E ? z[e] : -INFINITY;
+            sc[i] = e < E ? logit(e) : -INFINITY;
             zmax = fmaxf(zmax, sc[i]);
         }
         zmax = warp_max(zmax);
@@ -51,7 +52,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ z, const flo
 #pragma unroll
     for (int i = 0; i < kMaxExpertsPerLane; ++i) {
         const int e = lane + 32 * i;
-        sc[i] = e < E ? (ro.topk_softmax ? z[e] : (ro.softmax ? sc[i] * zsum : sigmoid_f(z[e]))) : 0.f;
+        sc[i] = e < E ? (ro.softmax ? sc[i] * zsum : (ro.topk_softmax ? logit(e) : sigmoid_f(logit(e)))) : 0.f;
         ch[i] = e < E ? sc[i] + (correction ? correction[e] : 0.f) : -INFINITY;
     }
     if (ro.groups > 0) {
@@ -228,22 +229,6 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const uint4* __restrict
     for (int c = threadIdx.x; c < n16; c += blockDim.x) out[(size_t)blockIdx.x * ld_out16 + c] = in[(size_t)r * ld_in16 + c];
 }
 
-template <typename T>
-__global__ void moe_combine_kernel(const T* __restrict__ eo, int ld_eo, const int* __restrict__ pos, const float* __restrict__ weight,
-                                   int top, const T* __restrict__ so, int ld_so, const float* __restrict__ shared_gate,
-                                   T* __restrict__ out, int ld_out, int W) {
-    const int r = blockIdx.x;
-    for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        float acc = 0.f;
-        for (int k = 0; k < top; ++k) {
-            const int p = pos[(size_t)r * top + k];
-            if (p >= 0) acc = fmaf(weight[(size_t)r * top + k], ldf(eo + (size_t)p * ld_eo + c), acc);
-        }
-        if (so) acc = fmaf(shared_gate ? shared_gate[r] : 1.f, ldf(so + (size_t)r * ld_so + c), acc);
-        stf(out + (size_t)r * ld_out + c, acc);
-    }
-}
-
 }  // namespace
 
 // a router's options are consistent with its sizes
@@ -295,19 +280,6 @@ int moe_gather_rows(int dt, const void* in, int ld_in, const int* src_row, void*
         return -2;
     count_launch();
     moe_gather_kernel<<<rows, 128, 0, s>>>((const uint4*)in, ld_in / per16, src_row, (uint4*)out, ld_out / per16, W / per16);
-    return cudaGetLastError() == cudaSuccess ? 0 : -100;
-}
-
-int moe_combine(int dt, const void* eo, int ld_eo, const int* pos, const float* weight, int top, const void* so, int ld_so,
-                const float* shared_gate, void* out, int ld_out, int S, int W, cudaStream_t s) {
-    if (!eo || !pos || !weight || !out || S < 1 || W < 1 || top < 1) return -2;
-    count_launch();
-    if (dt == DT_F32)
-        moe_combine_kernel<float><<<S, 256, 0, s>>>((const float*)eo, ld_eo, pos, weight, top, (const float*)so, ld_so, shared_gate,
-                                                    (float*)out, ld_out, W);
-    else
-        moe_combine_kernel<bf16><<<S, 256, 0, s>>>((const bf16*)eo, ld_eo, pos, weight, top, (const bf16*)so, ld_so, shared_gate,
-                                                   (bf16*)out, ld_out, W);
     return cudaGetLastError() == cudaSuccess ? 0 : -100;
 }
 

@@ -21,6 +21,27 @@ __device__ __forceinline__ bool seq_done(const SeqPos& p) { return p.finished &&
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 
+template <typename T> __device__ __forceinline__ void ld4(const T* p, float (&v)[4]);
+template <> __device__ __forceinline__ void ld4<float>(const float* p, float (&v)[4]) {
+    const float4 u = *reinterpret_cast<const float4*>(p);
+    v[0] = u.x; v[1] = u.y; v[2] = u.z; v[3] = u.w;
+}
+template <> __device__ __forceinline__ void ld4<bf16>(const bf16* p, float (&v)[4]) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+template <typename T> __device__ __forceinline__ void st4(T* p, const float (&v)[4]);
+template <> __device__ __forceinline__ void st4<float>(float* p, const float (&v)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+template <> __device__ __forceinline__ void st4<bf16>(bf16* p, const float (&v)[4]) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+}
+
+// choices of a routed row that a row kernel keeps in shared memory
+constexpr int kCombineTop = 32;
+
 template <typename T>
 __global__ void embed_sinusoid_kernel(const int64_t* __restrict__ ids, const int* __restrict__ seq_len, const T* __restrict__ table,
                                       int64_t vocab, float scale, const float* __restrict__ inv_freq, float* __restrict__ x32,
@@ -42,8 +63,8 @@ __global__ void embed_sinusoid_kernel(const int64_t* __restrict__ ids, const int
     }
 }
 
-// One CTA per row. Rows of up to 256 * kRowCache elements are read once into registers (E per thread, every load in flight
-// together); wider rows (E = 0) are re-read from L1/L2 in each of the three passes. Every form adds in the same order.
+// Two normed branches, averaged, behind a post-norm residual: one CTA per row. Rows of up to 256 * kRowCache elements are read once
+// into registers (E per thread, every load in flight together); wider rows (E = 0) are re-read from L1/L2 in each of the three passes. Every form adds in the same order.
 constexpr int kRowCache = 16;
 template <typename T, int E>
 __global__ void __launch_bounds__(256) postnorm_residual_kernel(float* __restrict__ x32, T* __restrict__ xa, const T* __restrict__ a,
@@ -54,7 +75,7 @@ __global__ void __launch_bounds__(256) postnorm_residual_kernel(float* __restric
     const int r = blockIdx.x;
     float* x = x32 + (size_t)r * W;
     const T* ar = a + (size_t)r * ld_a;
-    const T* br = b ? b + (size_t)r * ld_b : nullptr;
+    const T* br = b + (size_t)r * ld_b;
     constexpr bool CACHE = E > 0;
     constexpr int EN = E > 0 ? E : 1;
     float va[EN], vb[EN], vx[EN];
@@ -63,42 +84,38 @@ __global__ void __launch_bounds__(256) postnorm_residual_kernel(float* __restric
         for (int i = 0; i < EN; ++i) {
             const int c = threadIdx.x + i * 256;
             va[i] = c < W ? ldf(ar + c) : 0.f;
-            vb[i] = (br && c < W) ? ldf(br + c) : 0.f;
+            vb[i] = c < W ? ldf(br + c) : 0.f;
             vx[i] = c < W ? x[c] : 0.f;
         }
     }
-    float ra = 1.f, rb = 1.f;
-    if (br) {
-        float sa = 0.f, sb = 0.f;
-        if (CACHE) {
+    float sa = 0.f, sb = 0.f;
+    if (CACHE) {
 #pragma unroll
-            for (int i = 0; i < EN; ++i) { sa = fmaf(va[i], va[i], sa); sb = fmaf(vb[i], vb[i], sb); }
-        } else {
-            for (int c = threadIdx.x; c < W; c += blockDim.x) {
-                const float ta = ldf(ar + c), tb = ldf(br + c);
-                sa = fmaf(ta, ta, sa);
-                sb = fmaf(tb, tb, sb);
-            }
+        for (int i = 0; i < EN; ++i) { sa = fmaf(va[i], va[i], sa); sb = fmaf(vb[i], vb[i], sb); }
+    } else {
+        for (int c = threadIdx.x; c < W; c += blockDim.x) {
+            const float ta = ldf(ar + c), tb = ldf(br + c);
+            sa = fmaf(ta, ta, sa);
+            sb = fmaf(tb, tb, sb);
         }
-        sa = block_sum(sa, red);
-        sb = block_sum(sb, red);
-        ra = 1.f / sqrtf(sa / (float)W + eps);
-        rb = 1.f / sqrtf(sb / (float)W + eps);
     }
+    sa = block_sum(sa, red);
+    sb = block_sum(sb, red);
+    const float ra = 1.f / sqrtf(sa / (float)W + eps), rb = 1.f / sqrtf(sb / (float)W + eps);
     float ss = 0.f;
     if (CACHE) {
 #pragma unroll
         for (int i = 0; i < EN; ++i) {
             const int c = threadIdx.x + i * 256;
             if (c < W) {
-                const float m = br ? 0.5f * (va[i] * ra * wa[c] + vb[i] * rb * wb[c]) : va[i];
+                const float m = 0.5f * (va[i] * ra * wa[c] + vb[i] * rb * wb[c]);
                 vx[i] = fmaf(alpha, vx[i], m);
                 ss = fmaf(vx[i], vx[i], ss);
             }
         }
     } else {
         for (int c = threadIdx.x; c < W; c += blockDim.x) {
-            const float m = br ? 0.5f * (ldf(ar + c) * ra * wa[c] + ldf(br + c) * rb * wb[c]) : ldf(ar + c);
+            const float m = 0.5f * (ldf(ar + c) * ra * wa[c] + ldf(br + c) * rb * wb[c]);
             const float v = fmaf(alpha, x[c], m);
             ss = fmaf(v, v, ss);
         }
@@ -117,10 +134,111 @@ __global__ void __launch_bounds__(256) postnorm_residual_kernel(float* __restric
         }
     } else {
         for (int c = threadIdx.x; c < W; c += blockDim.x) {
-            const float m = br ? 0.5f * (ldf(ar + c) * ra * wa[c] + ldf(br + c) * rb * wb[c]) : ldf(ar + c);
+            const float m = 0.5f * (ldf(ar + c) * ra * wa[c] + ldf(br + c) * rb * wb[c]);
             const float v = fmaf(alpha, x[c], m) * rn * w[c];
             x[c] = v;
             stf(xa + (size_t)r * W + c, v);
+        }
+    }
+}
+
+// One branch behind a post-norm residual: x <- rms(alpha * x + ls * y) * w, one CTA per row; y = the sublayer's row, or the routed
+// feed-forward's weighted sum of expert rows. ls: a factor per column, or null. The new row stays in registers between its sum of
+// squares and its store (E pieces of V columns per thread; E = 0: rows wider than 256 * 16 pieces keep it in x32). A column's sum runs in
+// the same order for every S.
+template <typename T, int E, bool VEC>
+__global__ void __launch_bounds__(256) postnorm_branch_kernel(float* __restrict__ x32, T* __restrict__ xa, const T* __restrict__ a, int ld_a,
+                                                              bool has_mc, MoeCombine mc, const float* __restrict__ ls,
+                                                              const float* __restrict__ w, float alpha, float eps, int W) {
+    __shared__ float red[32];
+    __shared__ int spos[kCombineTop];
+    __shared__ float swt[kCombineTop];
+    constexpr int V = VEC ? 4 : 1, EN = E > 0 ? E : 1;
+    const int r = blockIdx.x;
+    float* x = x32 + (size_t)r * W;
+    const int top = has_mc ? mc.top : 0;
+    const bool cached = top <= kCombineTop;
+    float vx[EN][V];
+    if (E > 0) {            // the residual row's loads fly while the routed row's places are read
+#pragma unroll
+        for (int i = 0; i < EN; ++i) {
+            const int c = (threadIdx.x + i * 256) * V;
+#pragma unroll
+            for (int u = 0; u < V; ++u) vx[i][u] = 0.f;
+            if (c < W) { if (VEC) ld4(x + c, (float(&)[4])vx[i]); else vx[i][0] = x[c]; }
+        }
+    }
+    if (has_mc && cached) {
+        if (threadIdx.x < top) {
+            spos[threadIdx.x] = mc.pos[(size_t)r * top + threadIdx.x];
+            swt[threadIdx.x] = mc.weight[(size_t)r * top + threadIdx.x];
+        }
+        __syncthreads();
+    }
+    const float gs = (has_mc && mc.so) ? (mc.gate ? mc.gate[r] : 1.f) : 0.f;
+    auto add_branch = [&](int c, float (&v)[V]) {
+        float y[V], t[V];
+        if (!has_mc) {
+            if (VEC) ld4(a + (size_t)r * ld_a + c, (float(&)[4])y); else y[0] = ldf(a + (size_t)r * ld_a + c);
+        } else {
+#pragma unroll
+            for (int i = 0; i < V; ++i) y[i] = 0.f;
+            for (int k = 0; k < top; ++k) {
+                const int p = cached ? spos[k] : mc.pos[(size_t)r * top + k];
+                if (p < 0) continue;
+                const float wk = cached ? swt[k] : mc.weight[(size_t)r * top + k];
+                const T* src = (const T*)mc.eo + (size_t)p * mc.ld_eo + c;
+                if (VEC) ld4(src, (float(&)[4])t); else t[0] = ldf(src);
+#pragma unroll
+                for (int i = 0; i < V; ++i) y[i] = fmaf(wk, t[i], y[i]);
+            }
+            if (mc.so) {
+                const T* src = (const T*)mc.so + (size_t)r * mc.ld_so + c;
+                if (VEC) ld4(src, (float(&)[4])t); else t[0] = ldf(src);
+#pragma unroll
+                for (int i = 0; i < V; ++i) y[i] = fmaf(gs, t[i], y[i]);
+            }
+        }
+        if (ls) { if (VEC) ld4(ls + c, (float(&)[4])t); else t[0] = ls[c]; }
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] = fmaf(alpha, v[i], ls ? y[i] * t[i] : y[i]);
+    };
+    float ss = 0.f;
+    if (E > 0) {
+#pragma unroll
+        for (int i = 0; i < EN; ++i) {
+            const int c = (threadIdx.x + i * 256) * V;
+            if (c < W) add_branch(c, vx[i]);
+#pragma unroll
+            for (int u = 0; u < V; ++u) ss = fmaf(vx[i][u], vx[i][u], ss);
+        }
+    } else {
+        for (int c = threadIdx.x * V; c < W; c += 256 * V) {
+            float v[V];
+            if (VEC) ld4(x + c, (float(&)[4])v); else v[0] = x[c];
+            add_branch(c, v);
+#pragma unroll
+            for (int u = 0; u < V; ++u) ss = fmaf(v[u], v[u], ss);
+            if (VEC) st4(x + c, (const float(&)[4])v); else x[c] = v[0];
+        }
+    }
+    const float rn = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+    auto store = [&](int c, const float (&v)[V]) {
+        float o[V], t[V];
+        if (VEC) ld4(w + c, (float(&)[4])t); else t[0] = w[c];
+#pragma unroll
+        for (int u = 0; u < V; ++u) o[u] = v[u] * rn * t[u];
+        if (VEC) st4(x + c, (const float(&)[4])o); else x[c] = o[0];
+        if (VEC) st4(xa + (size_t)r * W + c, (const float(&)[4])o); else stf(xa + (size_t)r * W + c, o[0]);
+    };
+    if (E > 0) {
+#pragma unroll
+        for (int i = 0; i < EN; ++i) { const int c = (threadIdx.x + i * 256) * V; if (c < W) store(c, vx[i]); }
+    } else {
+        for (int c = threadIdx.x * V; c < W; c += 256 * V) {
+            float v[V];
+            if (VEC) ld4(x + c, (float(&)[4])v); else v[0] = x[c];
+            store(c, v);
         }
     }
 }
@@ -251,30 +369,11 @@ __global__ void __launch_bounds__(256) gather_norm_kernel(const float* __restric
     for (int c = threadIdx.x; c < W; c += blockDim.x) stf(out + (size_t)i * W + c, norm_apply(n, x[c] - mean, rn, c));
 }
 
-template <typename T> __device__ __forceinline__ void ld4(const T* p, float (&v)[4]);
-template <> __device__ __forceinline__ void ld4<float>(const float* p, float (&v)[4]) {
-    const float4 u = *reinterpret_cast<const float4*>(p);
-    v[0] = u.x; v[1] = u.y; v[2] = u.z; v[3] = u.w;
-}
-template <> __device__ __forceinline__ void ld4<bf16>(const bf16* p, float (&v)[4]) {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
-    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
-}
-template <typename T> __device__ __forceinline__ void st4(T* p, const float (&v)[4]);
-template <> __device__ __forceinline__ void st4<float>(float* p, const float (&v)[4]) {
-    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-}
-template <> __device__ __forceinline__ void st4<bf16>(bf16* p, const float (&v)[4]) {
-    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
-}
-
 // One CTA per row: pass 1 forms the new residual row (every addend read, also a row of xa that pass 2 rewrites) and, for a
 // norm with a row statistic, its sum of squares; pass 2 writes the normed row. The places and weights of a routed row's
 // choices are read once into shared memory, so that the expert rows' loads do not wait on them one by one. VEC: four
 // columns per thread and step (every row start 16-byte aligned in fp32, 8-byte in bf16). Each column's sum is formed in the
 // same order in both forms and does not depend on S.
-constexpr int kCombineTop = 32;
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) residual_norm_kernel(float* __restrict__ x32, const T* __restrict__ a, int ld_a,
                                                             const T* __restrict__ b, int ld_b, bool has_mc, MoeCombine mc, NormSpec n,
@@ -608,9 +707,34 @@ int embed_sinusoid(int dt, const int64_t* ids, const int* seq_len, const void* t
 }
 
 int postnorm_residual(int dt, float* x32, void* xa, const void* a, int ld_a, const float* wa, const void* b, int ld_b,
-                      const float* wb, const float* w, float alpha, float eps, int S, int W, cudaStream_t s) {
-    if (!x32 || !xa || !a || !w || S < 1 || W < 1 || (b && (!wa || !wb))) return -2;
+                      const float* wb, const float* w, float alpha, float eps, int S, int W, cudaStream_t s, const float* ls,
+                      const MoeCombine* mc) {
+    if (!x32 || !xa || (!a && !mc) || (a && mc) || !w || S < 1 || W < 1 || (b && (!wa || !wb || ls || mc))) return -2;
+    if (mc && (!mc->eo || !mc->pos || !mc->weight || mc->top < 1)) return -2;
     count_launch();
+    if (!b) {
+        const MoeCombine m = mc ? *mc : MoeCombine{};
+        const size_t es = dt == DT_F32 ? 4 : 2;
+        auto ok4 = [&](const void* p, int ld) { return !p || ((ld % 4) == 0 && ((uintptr_t)p % (4 * es)) == 0); };
+        const bool vec = (W % 4) == 0 && (((uintptr_t)x32 | (uintptr_t)w | (uintptr_t)ls) % 16) == 0 && ok4(a, ld_a) && ok4(xa, W) &&
+                         (!mc || (ok4(m.eo, m.ld_eo) && ok4(m.so, m.ld_so)));
+#define LCC_PNB2(E, VECB)                                                                                                      \
+    do {                                                                                                                       \
+        if (dt == DT_F32) postnorm_branch_kernel<float, E, VECB><<<S, 256, 0, s>>>(x32, (float*)xa, (const float*)a, ld_a, mc != nullptr, m, ls, w, alpha, eps, W); \
+        else postnorm_branch_kernel<bf16, E, VECB><<<S, 256, 0, s>>>(x32, (bf16*)xa, (const bf16*)a, ld_a, mc != nullptr, m, ls, w, alpha, eps, W);                 \
+    } while (0)
+#define LCC_PNB(E) do { if (vec) LCC_PNB2(E, true); else LCC_PNB2(E, false); } while (0)
+        const int pieces = (W / (vec ? 4 : 1) + 255) / 256;      // per thread: the form depends on the row's width alone
+        if (pieces <= 1) LCC_PNB(1);
+        else if (pieces <= 2) LCC_PNB(2);
+        else if (pieces <= 4) LCC_PNB(4);
+        else if (pieces <= 8) LCC_PNB(8);
+        else if (pieces <= kRowCache) LCC_PNB(16);
+        else LCC_PNB(0);
+#undef LCC_PNB
+#undef LCC_PNB2
+        return done();
+    }
 #define LCC_PNR(E)                                                                                                          \
     do {                                                                                                                    \
         if (dt == DT_F32)                                                                                                   \

@@ -72,13 +72,15 @@ Dims dims_of(const lcc_seq_layer& L) {
         z.a_kv = L.a_kv_from >= 0 ? 0 : z.a_kd;
         z.a_qin = L.a_q_rank > 0 ? L.a_q_rank : z.a_nq;
         z.a_gate = z.a_qin + z.a_kv;
-        z.a_proj = z.a_gate + (L.a_gate ? L.a_heads : 0);
+        if (L.a_gate == LCC_GATE_CHANNEL) z.a_gate = (z.a_gate + 7) / 8 * 8;     // (a tensor-core epilogue reads the gate block)
+        z.a_proj = z.a_gate + (L.a_gate == LCC_GATE_CHANNEL ? L.a_heads * L.a_vdim : (L.a_gate ? L.a_heads : 0));
         z.a_lat = L.a_heads * L.a_rank;
         z.a_o = L.a_heads * L.a_vdim;
     } else if (L.type == LCC_MIX_ATTENTION) {
         const int maps = L.m_maps > 1 ? L.m_maps : 1;
-        z.m_nq = L.m_heads * maps * L.m_dim; z.m_nk = L.m_kv_heads * maps * L.m_dim;
-        z.m_nv = L.m_value_keys ? 0 : L.m_kv_heads * L.m_vdim;
+        const bool own_kv = L.m_kv_from < 0;
+        z.m_nq = L.m_heads * maps * L.m_dim; z.m_nk = own_kv ? L.m_kv_heads * maps * L.m_dim : 0;
+        z.m_nv = L.m_value_keys || !own_kv ? 0 : L.m_kv_heads * L.m_vdim;
         z.m_vcol = L.m_value_keys ? z.m_nq : z.m_nq + z.m_nk;       // the values are the key columns as projected, or their own
         z.m_gate = z.m_nq + z.m_nk + z.m_nv;
         z.m_ngate = L.m_gate == LCC_GATE_CHANNEL ? L.m_heads * L.m_vdim : (L.m_gate == LCC_GATE_HEAD ? L.m_heads : 0);
@@ -239,15 +241,17 @@ int linear(const lcc_seq_model* m, const void* x, int ldx, const void* W, const 
 }
 
 // Per-head products: head h multiplies columns h * a_stride .. of x with the h-th [N, K] matrix of W and writes columns
-// h * c_stride .. of y. One batched tensor-core GEMM when the shapes allow it, else the grouped CUDA-core kernels.
+// h * c_stride .. of y. One batched tensor-core GEMM when the shapes allow it, else the grouped CUDA-core kernels. gate: rows of
+// gate logits laid out as y; every element of y is multiplied by their sigmoid.
 int linear_heads(const lcc_seq_model* m, const void* x, int ldx, int a_stride, const void* W, void* y, int ldy, int c_stride,
-                 bool y_f32, int heads, int M, int N, int K, cudaStream_t s) {
+                 bool y_f32, int heads, int M, int N, int K, cudaStream_t s, const void* gate = nullptr, int ld_gate = 0) {
     if (m->use_tc && m->d.dtype == LCC_DT_BF16 && M >= 16 && N >= 32 && (K % 64) == 0 && (N % 8) == 0 && (ldx % 8) == 0 &&
-        (ldy % 8) == 0 && (a_stride % 8) == 0 && (c_stride % 8) == 0) {
+        (ldy % 8) == 0 && (a_stride % 8) == 0 && (c_stride % 8) == 0 && (!gate || (!y_f32 && (ld_gate % 8) == 0 && ((uintptr_t)gate % 16) == 0))) {
         lcc::GemmArgs a;
         a.A = x; a.B = W; a.C = y; a.M = M; a.N = N; a.K = K; a.lda = ldx; a.ldb = K; a.ldc = ldy;
         a.bias = nullptr; a.residual = nullptr; a.ldr = 0; a.epi = lcc::EPI_NONE; a.block_n = 0;
         a.batch = heads; a.a_col_stride = a_stride; a.c_col_stride = c_stride; a.c_f32 = y_f32;
+        if (gate) { a.epi = lcc::EPI_SIGMOID_GATE; a.residual = gate; a.ldr = ld_gate; }
         return lcc::gemm_bf16_tn(a, m->ctx->num_sms, s);
     }
     lcc::GroupedLinear g{};
@@ -255,6 +259,29 @@ int linear_heads(const lcc_seq_model* m, const void* x, int ldx, int a_stride, c
     g.W = W; g.ldw = K; g.w_stride = (int64_t)N * K;
     g.C = y; g.ldc = ldy; g.c_stride = c_stride; g.c_f32 = y_f32;
     g.groups = heads; g.M = M; g.N = N; g.K = K;
+    g.gate = gate; g.ld_gate = ld_gate; g.gate_stride = c_stride;
+    return lcc::linear_grouped(g, s);
+}
+
+// h = clamped gated activation of [gate; up] W x: gate and up rows interleaved in groups of 16 (il16) form it in the product's epilogue or
+// store; otherwise large products leave the raw columns in `raw` and a row kernel follows.
+int linear_clamp_glu(const lcc_seq_model* m, const void* x, int ldx, const void* W, void* raw, int ldr, void* h, int ldh, float limit,
+                     bool il16, int M, int F, int K, cudaStream_t s) {
+    const bool tc = m->use_tc && m->d.dtype == LCC_DT_BF16 && M >= 16 && F >= 32 && K >= 64 && (K % 8) == 0 && (F % 8) == 0 && (ldx % 8) == 0 &&
+                    (ldh % 8) == 0 && (ldr % 8) == 0;
+    if (tc) {
+        lcc::GemmArgs a;
+        a.A = x; a.B = W; a.C = il16 ? h : raw; a.M = M; a.N = 2 * F; a.K = K; a.lda = ldx; a.ldb = K; a.ldc = il16 ? ldh : ldr;
+        a.bias = nullptr; a.residual = nullptr; a.ldr = 0; a.block_n = 0;
+        a.epi = il16 ? lcc::EPI_CLAMP_GLU : lcc::EPI_NONE;
+        a.epi_param = limit;
+        const int rc = lcc::gemm_bf16_tn(a, m->ctx->num_sms, s);
+        return rc || il16 ? rc : lcc::glu_clamp_swish(m->d.dtype, raw, ldr, h, ldh, M, F, limit, s);
+    }
+    lcc::GroupedLinear g{};
+    g.dt = m->d.dtype; g.A = x; g.lda = ldx; g.W = W; g.ldw = K; g.C = h; g.ldc = ldh;
+    g.groups = 1; g.M = M; g.N = F; g.K = K;
+    g.glu_F = F; g.glu_il16 = il16; g.glu_limit = limit; g.glu_tmp = raw; g.ld_tmp = ldr;
     return lcc::linear_grouped(g, s);
 }
 
@@ -292,8 +319,8 @@ lcc_seq_model* lcc_seq_model_create(lcc_ctx* ctx, const lcc_seq_model_desc* desc
             if (l.e_groups < 0 || (l.e_groups > 0 && (outs % l.e_groups || l.e_keep < 1 || l.e_keep > l.e_groups || l.e_keep * (outs / l.e_groups) < l.e_top)))
                 return fail("routed feed-forward: the kept groups must be equal groups that hold at least `top` experts");
             if (l.e_router_kind != LCC_ROUTER_SIGMOID && l.e_router_kind != LCC_ROUTER_SOFTMAX && l.e_router_kind != LCC_ROUTER_TOPK_SOFTMAX) return fail("unknown router kind");
-            if (l.e_router_kind == LCC_ROUTER_TOPK_SOFTMAX && (l.e_identity > 0 || l.e_groups > 0 || l.e_shared_ff > 0))
-                return fail("routed feed-forward: weights over the chosen logits combine with neither identity experts, groups nor a shared expert");
+            if (l.e_router_kind == LCC_ROUTER_TOPK_SOFTMAX && (l.e_identity > 0 || l.e_groups > 0))
+                return fail("routed feed-forward: weights over the chosen logits combine with neither identity experts nor groups");
             if (l.e_group_top < 0 || l.e_group_top > 2) return fail("routed feed-forward: a group scores as its best one or two scores");
             if (l.e_act < LCC_EXPERT_RELU2 || l.e_act > LCC_EXPERT_GELU) return fail("unknown expert activation");
             if (l.e_up_il16 && (l.e_act == LCC_EXPERT_RELU2 || l.e_act == LCC_EXPERT_GELU || l.e_ff % 16)) return fail("interleaved gate / up rows need a gated expert width that is a multiple of 16");
@@ -303,10 +330,13 @@ lcc_seq_model* lcc_seq_model_create(lcc_ctx* ctx, const lcc_seq_model_desc* desc
         if (bn && l.canon_w_f32 && desc->canon_taps < 1) return fail("a convolution in front of the mixer needs its tap count");
         if (!l.norm1_f32 || (l.ff > 0 && ((!par && !l.norm2_f32) || !l.ff_in || !l.ff_out))) return fail("missing norm / feed-forward weights");
         if (sw && (!l.norm1b_f32 || ((l.ff > 0 || l.ff_kind == LCC_FF_MOE) && !l.norm2b_f32))) return fail("missing norms behind the sublayers");
+        if (l.ff_kind == LCC_FF_GLU && l.ff > 0 && l.ff_act != LCC_ACT_GELU_TANH && l.ff_act != LCC_ACT_CLAMP_GLU) return fail("unknown gated feed-forward activation");
+        if (l.ff_il16 && (l.ff_kind != LCC_FF_GLU || l.ff_act != LCC_ACT_CLAMP_GLU || l.ff % 16)) return fail("interleaved gate / up rows need the clamped form and a width that is a multiple of 16");
+        if ((l.ls1_f32 || l.ls2_f32) && (desc->block != LCC_BLOCK_POSTNORM || l.type == LCC_MIX_PARALLEL)) return fail("factors on the sublayers' outputs are served in post-norm blocks with one branch");
         if (l.ff_kind == LCC_FF_MLP && l.ff_act != LCC_ACT_GELU_TANH && l.ff_act != LCC_ACT_RELU2) return fail("unknown feed-forward activation");
         if (dyt && !l.norm1_bias_f32) return fail("missing norm bias");
         if (par && l.type != LCC_MIX_ATTENTION) return fail("a parallel block takes the attention mixer");
-        if (!par && !bn && !sw && l.type == LCC_MIX_ATTENTION) return fail("the attention mixer is not served in post-norm blocks and blocks on several streams");
+        if (hc && l.type == LCC_MIX_ATTENTION) return fail("the attention mixer is not served in blocks on several streams");
         if ((bn || sw) && l.type == LCC_MIX_PARALLEL) return fail("the parallel mixer merges its branches in a post-norm block");
         if (hc && (!l.hc1_f32 || ((l.ff > 0 || l.ff_kind == LCC_FF_MOE) && !l.hc2_f32))) return fail("missing stream weights");
         if (hc && l.type == LCC_MIX_PARALLEL) return fail("the parallel mixer merges its branches in a post-norm block");
@@ -341,7 +371,7 @@ lcc_seq_model* lcc_seq_model_create(lcc_ctx* ctx, const lcc_seq_model_desc* desc
             }
             if (!l.a_in || !l.a_uk_t || !l.a_uv || !l.a_out || !l.rot_inv_freq_f32 || (l.a_q_rank > 0 && (!l.a_uq || !l.a_q_norm_f32)))
                 return fail("latent attention layer: missing weights");
-            if (l.a_q_rank < 0 || l.a_window < 0) return fail("latent attention layer: unsupported sizes");
+            if (l.a_q_rank < 0 || l.a_window < 0 || l.a_gate < LCC_GATE_NONE || l.a_gate > LCC_GATE_CHANNEL) return fail("latent attention layer: unsupported sizes");
         } else if (l.type == LCC_MIX_ATTENTION) {
             if (l.m_heads < 1 || l.m_kv_heads < 1 || l.m_heads % l.m_kv_heads || l.m_dim < 1 || l.m_vdim < 1 || l.m_rot_dims < 0 ||
                 (l.m_rot_dims & 1) || l.m_rot_dims > l.m_dim || (l.m_value_keys && l.m_vdim != l.m_dim) || l.m_gate < LCC_GATE_NONE ||
@@ -350,7 +380,15 @@ lcc_seq_model* lcc_seq_model_create(lcc_ctx* ctx, const lcc_seq_model_desc* desc
             if (l.m_maps < 0 || l.m_maps > 2 || l.m_keep_first < 0 || (l.m_keep_first > 0 && l.m_chunk > 0) ||
                 (l.m_maps == 2 && (l.m_value_keys || l.m_gate != LCC_GATE_NONE || l.m_sink || l.m_rot_dims || !l.m_no_qk_norm || l.m_unit_norm || l.m_temp_f32)))
                 return fail("attention layer: unsupported options (two maps combine with projected values only: no norm, rotation, gate or sink)");
-            if (!l.m_in || (!l.m_unit_norm && !l.m_no_qk_norm && (!l.m_qnorm_f32 || !l.m_knorm_f32)) || !l.m_out || (l.m_rot_dims > 0 && !l.rot_inv_freq_f32))
+            if (l.m_kv_from >= 0) {
+                if (l.m_kv_from >= i) return fail("attention layer: the shared cache must belong to an earlier layer");
+                const lcc_seq_layer& o = desc->layers[l.m_kv_from];
+                if (o.type != LCC_MIX_ATTENTION || o.m_kv_from >= 0 || o.m_kv_heads != l.m_kv_heads || o.m_dim != l.m_dim || o.m_vdim != l.m_vdim ||
+                    l.m_maps == 2 || o.m_maps == 2 || l.m_value_keys || l.m_vmix_role || l.m_in_bias_f32)
+                    return fail("attention layer: the shared cache has another geometry");
+            }
+            if (l.m_temp_every < 0 || (l.m_bias_f32 && l.m_bias_len < 1)) return fail("attention layer: unsupported query temperature or bias table");
+            if (!l.m_in || (!l.m_unit_norm && !l.m_no_qk_norm && (!l.m_qnorm_f32 || (!l.m_knorm_f32 && l.m_kv_from < 0))) || !l.m_out || (l.m_rot_dims > 0 && !l.rot_inv_freq_f32))
                 return fail("attention layer: missing weights");
             if (l.m_vmix_role < 0 || l.m_vmix_role > 2 || (l.m_vmix_role && l.m_value_keys)) return fail("attention layer: values are mixed across layers only when they are projected");
             if (l.m_vmix_role == 1) {
@@ -622,7 +660,7 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
                 STEP(lcc::latent_kv_append(dt, proj + ((size_t)r0 * ldp + (own_q ? z.a_qin : 0)) * es, ldp, l.a_kv_from < 0, l.a_latent_norm_f32, d.eps,
                                            l.rot_inv_freq_f32, l.rot_mag, q32 + (size_t)r0 * H * z.a_kd, en.k_pages[src], en.page_table,
                                            page_size, en.n_new, H, l.a_dim, l.a_rot_dim, l.a_rank, pos_of(en), s,
-                                           own_q ? qsrc + (size_t)r0 * ldq * es : nullptr, ldq), "latent cache append");
+                                           own_q ? qsrc + (size_t)r0 * ldq * es : nullptr, ldq, l.a_rot_pairs != 0), "latent cache append");
                 r0 += en.n_new;
             }
             STEP(linear_heads(m, qsrc, ldq, QH, l.a_uk_t, q32, H * z.a_kd, z.a_kd, true, H, T, l.a_rank, l.a_dim, s), "query absorption");
@@ -630,12 +668,14 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
             for (int e = 0; e < n_entries; ++e) {
                 const lcc_seq_entry& en = entries[e];
                 STEP(lcc::attn_masked(dt, q32 + (size_t)r0 * H * z.a_kd, en.k_pages[src], en.k_pages[src], en.page_table, page_size,
-                                      l.a_gate ? proj + ((size_t)r0 * ldp + z.a_gate) * es : nullptr, ldp, mid + (size_t)r0 * ldl * es, ldl, en.n_new, H, 1,
+                                      l.a_gate == LCC_GATE_HEAD ? proj + ((size_t)r0 * ldp + z.a_gate) * es : nullptr, ldp, mid + (size_t)r0 * ldl * es, ldl, en.n_new, H, 1,
                                       z.a_kd, l.a_rank, 0, l.a_scale, m->use_tc, pos_of(en), s, lo, l.a_sink_f32, z.a_kd, split_ws, L.split_floats,
                                       en.past + en.n_new), "latent attention");
                 r0 += en.n_new;
             }
-            STEP(linear_heads(m, mid, ldl, l.a_rank, l.a_uv, mid2, ldo, l.a_vdim, false, H, T, l.a_vdim, l.a_rank, s), "value up-projection");
+            // (a gate per channel multiplies the heads in the up-projection's store)
+            const uint8_t* vgate = l.a_gate == LCC_GATE_CHANNEL ? proj + (size_t)z.a_gate * es : nullptr;
+            STEP(linear_heads(m, mid, ldl, l.a_rank, l.a_uv, mid2, ldo, l.a_vdim, false, H, T, l.a_vdim, l.a_rank, s, vgate, ldp), "value up-projection");
             STEP(linear(m, mid2, ldo, l.a_out, nullptr, o1, W, false, T, W, z.a_o, s), "latent attention out-proj");
         } else if (l.type == LCC_MIX_ATTENTION) {
             // [q | k | (v) | gate] -> per-head q/k norm + rotary positions, k and the values (the key columns as projected, or
@@ -645,13 +685,16 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
             lcc::AttnOpts ao;
             ao.window = l.m_window; ao.no_sink = !l.m_sink; ao.gate_channel = l.m_gate == LCC_GATE_CHANNEL;
             ao.keep_first = l.m_keep_first; ao.softcap = l.m_softcap;
+            ao.bias = l.m_bias_f32; ao.bias_len = l.m_bias_len;
+            const bool own_kv = l.m_kv_from < 0;
+            const int src = own_kv ? li : l.m_kv_from;        // whose pages hold the keys and values
             const int maps = l.m_maps > 1 ? l.m_maps : 1;
             if (maps > 1) { ao.maps = maps; ao.lambda = l.m_lambda; ao.diff_scale = l.m_diff_scale; ao.eps = d.eps; }
             int r0 = 0;
             for (int e = 0; e < n_entries; ++e) {
                 const lcc_seq_entry& en = entries[e];
-                if (!en.k_pages || !en.v_pages || !en.k_pages[li] || !en.v_pages[li] || !en.page_table)
-                    LCC_FAIL(m->ctx, -2, "lcc_seq_forward: entry %d has no pages for layer %d", e, li);
+                if (!en.k_pages || !en.v_pages || !en.k_pages[src] || !en.v_pages[src] || !en.page_table)
+                    LCC_FAIL(m->ctx, -2, "lcc_seq_forward: entry %d has no pages for layer %d", e, src);
                 const lcc::SeqPos pos = pos_of(en);
                 uint8_t* pr = proj + (size_t)r0 * ldp * es;
                 float* q = q32 + (size_t)r0 * z.m_nq;
@@ -659,12 +702,12 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
                 const int ldk = ld8(z.m_nv);
                 const lcc::AppendOpts apo{l.m_unit_norm != 0, l.m_temp_f32,
                                           l.m_vmix_role == 2 ? vkeep + (size_t)r0 * ldk * es : nullptr, ldk, l.m_vmix,
-                                          l.m_vmix_role == 1 ? vkeep + (size_t)r0 * ldk * es : nullptr, ldk};
+                                          l.m_vmix_role == 1 ? vkeep + (size_t)r0 * ldk * es : nullptr, ldk, l.m_temp_coef, l.m_temp_every, !own_kv};
                 STEP(lcc::qk_headnorm_rope_append(dt, pr, ldp, z.m_vcol, l.m_qnorm_f32, l.m_knorm_f32, d.eps, l.rot_inv_freq_f32, l.rot_mag,
-                                                  l.m_rot_dims, l.m_rot_pairs, q, en.k_pages[li], en.v_pages[li], en.page_table, page_size,
+                                                  l.m_rot_dims, l.m_rot_pairs, q, en.k_pages[src], en.v_pages[src], en.page_table, page_size,
                                                   en.n_new, l.m_heads, l.m_kv_heads, maps * l.m_dim, l.m_vdim, pos, s, &apo), "q/k norm + rotary + cache append");
                 if (maps > 1) ao.raw = y32 + (size_t)r0 * l.m_heads * maps * l.m_vdim;
-                STEP(lcc::attn_masked(dt, q, en.k_pages[li], en.v_pages[li], en.page_table, page_size,
+                STEP(lcc::attn_masked(dt, q, en.k_pages[src], en.v_pages[src], en.page_table, page_size,
                                       z.m_ngate ? pr + (size_t)z.m_gate * es : nullptr, ldp, mid + (size_t)r0 * ldo * es, ldo, en.n_new,
                                       l.m_heads, l.m_kv_heads, l.m_dim, l.m_vdim, l.m_chunk, l.m_scale, m->use_tc, pos, s, ao, nullptr, 0,
                                       split_ws, L.split_floats, en.past + en.n_new), "window attention");
@@ -769,9 +812,9 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
             STEP(lcc::sandwich_residual(dt, x32, o1, W, nullptr, spec_of(l.norm1b_f32), has_ff ? spec_of(l.norm2_f32) : norm_of(li + 1), xa, T, W, s),
                  "norm1b + residual + next norm");
         else if (l.type != LCC_MIX_PARALLEL)
-            STEP(lcc::postnorm_residual(dt, x32, xa, o1, W, nullptr, nullptr, 0, nullptr, l.norm1_f32, d.alpha, d.eps, T, W, s), "norm1");
+            STEP(lcc::postnorm_residual(dt, x32, xa, o1, W, nullptr, nullptr, 0, nullptr, l.norm1_f32, d.alpha, d.eps, T, W, s, l.ls1_f32), "norm1");
         if (has_ff && hc) STEP(boundary(l.hc2_f32, l.norm2_f32, nullptr), "stream boundary");
-        lcc::MoeCombine par_mc{};       // parallel, output-normed and sandwich blocks: the routed feed-forward's row is formed by the layer's residual kernel
+        lcc::MoeCombine par_mc{};       // blocks on one stream: the routed feed-forward's row is formed by the layer's residual kernel
         bool par_is_mc = false;
         if (l.ff_kind == LCC_FF_MOE) {
             // E real experts own row lists; the router has EO = E + identity outputs
@@ -782,7 +825,7 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
             const int E = l.e_experts, EO = E + l.e_identity, K = l.e_top, lde = ld8(EO + 1), NH = glu ? 2 * l.e_ff : l.e_ff, ldh = ld8(NH),
                       ldg = ld8(l.e_ff), ldw8 = ld8(W), lds = ld8(l.e_shared_ff);
             const lcc::MoeRouterOpts ro{l.e_router_kind == LCC_ROUTER_SOFTMAX, l.e_identity, l.e_groups, l.e_keep, l.e_router_kind == LCC_ROUTER_TOPK_SOFTMAX,
-                                       l.e_group_top > 1 ? l.e_group_top : 1};
+                                       l.e_group_top > 1 ? l.e_group_top : 1, l.e_router_bias_f32};
             const int up_act = glu ? lcc::ACT_NONE : (l.e_act == LCC_EXPERT_GELU ? lcc::ACT_GELU_ERF : lcc::ACT_RELU2);
             float* mf = (float*)(ws + L.moe_f);
             float* logit = mf; float* wsel = mf + (size_t)T * lde; float* sgate = wsel + (size_t)T * K;
@@ -855,11 +898,9 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
             if (hc) {   // the weighted sum of the experts' rows is formed by the boundary kernel that folds it into the streams
                 pend_mc = lcc::MoeCombine{eo, ldw8, posn, wsel, K, shared ? o2 : nullptr, W, gate_out};
                 pend_is_mc = true;
-            } else if (par || bn || sw) {   // ... or by the residual kernel that closes the layer; identity experts return the normed row
+            } else {   // ... or by the residual kernel that closes the layer; identity experts return the normed row
                 par_mc = lcc::MoeCombine{eo, ldw8, posn, wsel, K, shared ? (const void*)o2 : (ident ? (const void*)xa : nullptr), W, gate_out};
                 par_is_mc = true;
-            } else {
-                STEP(lcc::moe_combine(dt, eo, ldw8, posn, wsel, K, shared ? o2 : nullptr, W, gate_out, o1, W, T, W, fs), "expert combine");
             }
         } else if (l.ff > 0 && l.ff_kind == LCC_FF_MLP) {
             const int ldf = ld8(l.ff);
@@ -869,8 +910,12 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
             STEP(linear(m, mid2, ldf, l.ff_out, nullptr, par ? o2 : o1, W, false, T, W, l.ff, fs), "feed-forward down");
         } else if (l.ff > 0) {
             const int ldg = ld8(2 * l.ff), ldf = ld8(l.ff);
-            STEP(linear(m, xa, W, l.ff_in, nullptr, proj, ldg, false, T, 2 * l.ff, W, fs), "feed-forward in");
-            STEP(lcc::glu_gelu_tanh(dt, proj, ldg, mid, ldf, T, l.ff, fs), "gated gelu");
+            if (l.ff_act == LCC_ACT_CLAMP_GLU) {
+                STEP(linear_clamp_glu(m, xa, W, l.ff_in, proj, ldg, mid, ldf, l.ff_limit, l.ff_il16 != 0, T, l.ff, W, fs), "feed-forward in + clamped gate");
+            } else {
+                STEP(linear(m, xa, W, l.ff_in, nullptr, proj, ldg, false, T, 2 * l.ff, W, fs), "feed-forward in");
+                STEP(lcc::glu_gelu_tanh(dt, proj, ldg, mid, ldf, T, l.ff, fs), "gated gelu");
+            }
             STEP(linear(m, mid, ldf, l.ff_out, nullptr, par ? o2 : o1, W, false, T, W, l.ff, fs), "feed-forward out");
         }
         if (fork_ff && (cudaEventRecord(m->ev_join, m->side) != cudaSuccess || cudaStreamWaitEvent(s, m->ev_join, 0) != cudaSuccess))
@@ -889,7 +934,8 @@ int lcc_seq_forward(lcc_seq_model* m, const lcc_seq_entry* entries, int n_entrie
                                         xa, T, W, s), "norm2b + residual + next norm");
         } else if (has_ff) {
             if (hc) pend_hc = l.hc2_f32;
-            else STEP(lcc::postnorm_residual(dt, x32, xa, o1, W, nullptr, nullptr, 0, nullptr, l.norm2_f32, d.alpha, d.eps, T, W, s), "norm2");
+            else STEP(lcc::postnorm_residual(dt, x32, xa, par_is_mc ? nullptr : o1, W, nullptr, nullptr, 0, nullptr, l.norm2_f32, d.alpha, d.eps, T, W, s,
+                                             l.ls2_f32, par_is_mc ? &par_mc : nullptr), "norm2");
         }
         if (layer_dump && !hc) {
             if (cudaMemcpyAsync(layer_dump + (size_t)li * T * W, x32, (size_t)T * W * 4, cudaMemcpyDeviceToDevice, s) != cudaSuccess)

@@ -7,7 +7,7 @@
 //   rotary.cu       rotate-half rotary positions on slices of a projection, packed to fp32 for a recurrence
 //   attn_latent.cu  latent (low-rank) K/V cache: latent norm + shared rotary key part -> pages, rotary query part
 //   hyper.cu        pre-norm blocks on several residual streams (hyper-connections)
-//   moe.cu          sigmoid, softmax or chosen-logit-softmax top-k router (groups of experts, identity experts), expert row lists, weighted combine
+//   moe.cu          sigmoid, softmax or chosen-logit-softmax top-k router (groups of experts, identity experts, logit biases), expert row lists
 // Every op exists for two storage types (DT_BF16: bf16 storage, fp32 arithmetic where the model asks for it;
 // DT_F32: everything fp32). All return 0 on success, negative on invalid arguments; launches are asynchronous on `s`.
 #pragma once
@@ -63,6 +63,8 @@ struct GroupedLinear {
     // the general gated activation g * sigmoid(alpha g) * (u + up_bias) with g = min(gate, limit), u = clamp(up, -limit, limit):
     // the defaults are the clamped form above; alpha 1, up_bias 0 and an infinite limit give silu(gate) * up
     float glu_alpha = 1.702f, glu_up_bias = 1.f;
+    // gate (storage dt; plain groups without lists, no GLU): C[r, c] of group z is multiplied by sigmoid(gate[r, z * gate_stride + c])
+    const void* gate = nullptr; int ld_gate = 0; int64_t gate_stride = 0;
 };
 enum { ACT_NONE = 0, ACT_RELU2 = 1, ACT_GELU_TANH = 2, ACT_GELU_ERF = 3 };   // 3: 0.5 x (1 + erf(x / sqrt(2))); 2: 0.5 x (1 + tanh(sqrt(2/pi) (x + 0.044715 x^3)))
 int linear_grouped(const GroupedLinear& g, cudaStream_t s);
@@ -198,6 +200,8 @@ size_t attn_split_ws_floats(int rows, int Hq, int DV);
 // q is [S, Hq, 2, D] and a K row holds the two maps of a key/value head (2 * D channels); each map is a softmax of its own over the
 // same values, and the head's output is rms(a1 - lambda * a2) * diff_scale over its DV channels (x / sqrt(mean(x^2) + eps)). raw: fp32
 // [S, Hq, 2, DV] scratch for the kernels that do not form the difference themselves (given with maps = 2 only).
+// bias: fp32 [heads][bias_len], added to a head's score behind the scale and the cap: entry d for a key d positions back, the last entry
+// for every key further away.
 struct AttnOpts {
     int window = 0;
     bool no_sink = false, gate_channel = false;
@@ -206,12 +210,21 @@ struct AttnOpts {
     int maps = 1;
     float lambda = 0.f, diff_scale = 1.f, eps = 0.f;
     float* raw = nullptr;
+    const float* bias = nullptr;
+    int bias_len = 0;
 };
 // Options of qk_headnorm_rope_append (null: none). unit_norm: q and k heads are divided by their rms without a weight (qn_w, kn_w
 // null; the rotation keeps every pair's length, so norming before it equals norming after it). q_head_scale: fp32 [Hq], one factor
 // per query head on q_out (a temperature on the scores). v_mix: [S, ld_mix] slice (storage dt) of G*DV columns: the cached values
-// are (1 - mix) * v + mix * v_mix in fp32. v_keep: [S, ld_keep] (storage dt) receives the values as projected.
-struct AppendOpts { bool unit_norm; const float* q_head_scale; const void* v_mix; int ld_mix; float mix; void* v_keep; int ld_keep; };
+// are (1 - mix) * v + mix * v_mix in fp32. v_keep: [S, ld_keep] (storage dt) receives the values as projected. temp_every > 0: the
+// queries at position p are multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1). q_only: the rows hold queries only (the
+// layer reads keys and values that another layer cached) and nothing is appended.
+struct AppendOpts {
+    bool unit_norm; const float* q_head_scale; const void* v_mix; int ld_mix; float mix; void* v_keep; int ld_keep;
+    float temp_coef = 0.f;
+    int temp_every = 0;
+    bool q_only = false;
+};
 int attn_masked(int dt, const float* q, const void* k_pages, const void* v_pages, const int* page_table, int page_size,
                 const void* gate, int ld_gate, void* out, int ld_out, int S, int Hq, int G, int D, int DV, int chunk, float scale,
                 bool tensor_cores, SeqPos pos, cudaStream_t s, const AttnOpts& opt, const float* sink = nullptr, int ld_v = 0,
@@ -246,10 +259,11 @@ int rotary_pack_f32(int dt, const void* in, int ld_in, float* out, int ld_out, c
 // at positions past .. past+S-1. Always: the rotated part of each head's query goes to q_out fp32 [S, H, R + DR] at
 // channels R .. R+DR-1 (channels 0 .. R-1 are left for the absorbed unrotated part: W_uk_h^T q_h).
 // q (optional): the query heads [S, ld_q] (storage dt) when they are not the first columns of proj (queries that come through
-// a latent of their own); proj then starts with the latent.
+// a latent of their own); proj then starts with the latent. rot_pairs: channel 2i of the rotated part turns with 2i+1, else i with
+// i + DR/2.
 int latent_kv_append(int dt, const void* proj, int ld, int has_kv, const float* norm_w, float eps, const float* inv_freq,
                      float mag, float* q_out, void* k_pages, const int* page_table, int page_size, int S, int H, int D,
-                     int DR, int R, SeqPos pos, cudaStream_t s, const void* q = nullptr, int ld_q = 0);
+                     int DR, int R, SeqPos pos, cudaStream_t s, const void* q = nullptr, int ld_q = 0, bool rot_pairs = false);
 
 // ---- hyper.cu -----------------------------------------------------------------------------------------------------------
 // One boundary between two sublayers of a pre-norm block on n residual streams xs fp32 [S, n, W]:
@@ -258,7 +272,7 @@ int latent_kv_append(int dt, const void* proj, int ld, int has_kv, const float* 
 //   (3) if sum_out: sum_out = sum_s x_s  (fp32 [S, W])
 // prev: fp32 [in: n | out: n | mix: n*n] of the sublayer that produced y; next: the same block of the sublayer that reads xa.
 // mc (instead of y): the finished sublayer is a routed feed-forward whose output row is formed here,
-//   y[r] = sum_k weight[r, k] * eo[pos[r, k]] + gate[r] * so[r]   (in fp32; moe_combine as part of the boundary).
+//   y[r] = sum_k weight[r, k] * eo[pos[r, k]] + gate[r] * so[r]   (in fp32).
 int hyper_boundary(int dt, float* xs, int n, const void* y, int ld_y, const float* prev, const float* next, const float* w,
                    float eps, void* xa, float* sum_out, int S, int W, cudaStream_t s, const MoeCombine* mc = nullptr);
 
@@ -274,9 +288,10 @@ int hyper_boundary(int dt, float* xs, int n, const void* y, int ld_y, const floa
 // must then be given; the logits have no shared-gate column); groups > 0: the E outputs form that many equal groups of
 // neighbours, a group scores as its largest choice score and only members of the `keep` best groups can be chosen.
 // topk_softmax: the choice is by logit (+ correction) and the weights are the softmax over the chosen logits only (times scale);
-// it combines with neither identity experts nor groups. correction may be null (zeros). group_top: a group scores as the sum of that
+// it combines with neither identity experts nor groups. correction may be null (zeros). logit_bias: fp32 [E], added to the logits
+// themselves before scores and choice (not to the shared gate's). group_top: a group scores as the sum of that
 // many of its largest choice scores (1 or 2).
-struct MoeRouterOpts { bool softmax; int identity; int groups; int keep; bool topk_softmax = false; int group_top = 1; };
+struct MoeRouterOpts { bool softmax; int identity; int groups; int keep; bool topk_softmax = false; int group_top = 1; const float* logit_bias = nullptr; };
 int moe_route(const float* logits, int ld, const float* correction, int E, int top, float scale, int* sel, float* weight,
               float* shared_gate, int* counts, int* rank, int S, cudaStream_t s, const MoeRouterOpts* opt = nullptr);
 // moe_route and moe_index (dense lists) in one launch of one CTA, for calls of up to kMoeSmallItems (row, choice) pairs; it
@@ -292,11 +307,6 @@ int moe_index(const int* sel, const int* rank, const int* counts, int E, int top
               int* tile_group, int n_tiles, int S, cudaStream_t s);
 // out[i, :] = in[src_row[i], :] for rows with src_row[i] >= 0 (storage dt; W, leading dimensions and bases 16-byte aligned)
 int moe_gather_rows(int dt, const void* in, int ld_in, const int* src_row, void* out, int ld_out, int rows, int W, cudaStream_t s);
-// out[r, :] = sum_k weight[r, k] * eo[pos[r, k], :] (+ shared_gate[r] * so[r, :])   (eo, so, out: storage dt); choices with
-// pos < 0 (identity experts) are skipped: their share is the so term
-int moe_combine(int dt, const void* eo, int ld_eo, const int* pos, const float* weight, int top, const void* so, int ld_so,
-                const float* shared_gate, void* out, int ld_out, int S, int W, cudaStream_t s);
-
 // ---- rowops.cu ----------------------------------------------------------------------------------------------------------
 // x[r, :] = table[id_r, :] * scale + sinusoid(past + r): entry 2i = sin(p * inv_freq[i]), 2i+1 = cos of the same
 // (inv_freq null: no position term). ids: device int64; when seq_len is non-null, row r reads ids[*seq_len - S + r].
@@ -304,9 +314,11 @@ int moe_combine(int dt, const void* eo, int ld_eo, const int* pos, const float* 
 int embed_sinusoid(int dt, const int64_t* ids, const int* seq_len, const void* table, int64_t vocab, float scale,
                    const float* inv_freq, float* x32, void* xa, int S, int W, SeqPos pos, cudaStream_t s, int copies = 1);
 // Post-norm residual block: m = a, or (two branches) m = (rms(a) * wa + rms(b) * wb) / 2; x <- rms(alpha * x + m) * w.
-// a, b: [S, W] (storage dt); wa, wb, w: fp32 [W]; x32 updated in place, xa = copy in storage dt.
+// a, b: [S, W] (storage dt); wa, wb, w: fp32 [W]; x32 updated in place, xa = copy in storage dt. One branch only: mc (instead of a)
+// forms the routed feed-forward's row here as in residual_norm; ls (fp32 [W], optional) multiplies the branch element by element.
 int postnorm_residual(int dt, float* x32, void* xa, const void* a, int ld_a, const float* wa, const void* b, int ld_b,
-                      const float* wb, const float* w, float alpha, float eps, int S, int W, cudaStream_t s);
+                      const float* wb, const float* w, float alpha, float eps, int S, int W, cudaStream_t s, const float* ls = nullptr,
+                      const MoeCombine* mc = nullptr);
 // Grouped RMS norm with a multiplicative silu gate: y: fp32 [S, n]; gate: [S, n] slice (storage dt). Groups of `group`
 // consecutive columns; weight w[c % w_len]. gate_first 1: out = rms(y * silu(g)) * w; 0: out = rms(y) * w * silu(g);
 // 2: out = rms(y) * w * sigmoid(g). group = n: one norm over the whole row.

@@ -26,6 +26,7 @@ register("Kedelorn", "livecc_b200.seq_engine", "SeqLMForCausalLM")
 register("Dibedra", "livecc_b200.seq_engine", "SeqLMForCausalLM")
 register("Lugizen", "livecc_b200.seq_engine", "SeqLMForCausalLM")
 register("Kapitar", "livecc_b200.seq_engine", "SeqLMForCausalLM")
+register("Poresun", "livecc_b200.seq_engine", "SeqLMForCausalLM")
 
 
 def architectures() -> list:

@@ -18,6 +18,7 @@ from __future__ import annotations
 
 import ctypes as C
 import json
+import math
 import os
 from typing import Dict, List, Optional, Sequence, Tuple
 
@@ -35,6 +36,23 @@ def _dtype_of(torch_dtype) -> torch.dtype:
     if torch_dtype in (torch.float32, "float32", "fp32", "float"):
         return torch.float32
     raise NotImplementedError(f"torch_dtype={torch_dtype!r}: the hybrid sequence models run in bfloat16 or float32")
+
+
+def distance_bias(rel: torch.Tensor, heads: int, far: float, name: str) -> torch.Tensor:
+    """Bias table `rel` [buckets, heads] -> fp32 [heads, n]: what a key d positions back adds to a head's score; the last entry holds for
+    every key further away. Distances below half the table have a bucket each, the other buckets grow geometrically up to `far`."""
+    if rel.dim() != 2 or rel.shape[1] != heads:
+        raise ValueError(f"{name} has shape {tuple(rel.shape)}, config.json implies [buckets, {heads}]")
+    rows = rel.shape[0]
+    half = rows // 2
+    if half < 1 or far <= half:
+        raise ValueError(f"{name}: {rows} buckets do not reach {far} positions")
+    idx, n = [], 0
+    while not idx or idx[-1] < rows - 1:
+        # (the small term keeps a distance whose logarithms meet an integer exactly from falling below it)
+        idx.append(n if n < half else min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half) + 1e-9)))
+        n += 1
+    return rel.to(torch.float32)[torch.tensor(idx, device=rel.device)].t().contiguous()
 
 
 class SeqWeights:
@@ -70,6 +88,10 @@ class SeqWeights:
                     raise ValueError(f"{name} is not a single number")
                 return f32(get(name).to(torch.float32).reshape(1).expand(cfg.width))
             return f32(get(name).to(torch.float32) + cfg.norm_offset) if cfg.norm_offset else f32(get(name))
+
+        def il16(g, u):   # gate and up rows interleaved in groups of 16: one product's neighbouring columns are a pair
+            n = g.shape[0]
+            return torch.stack([g.view(n // 16, 16, W), u.view(n // 16, 16, W)], 1).reshape(2 * n, W)
 
         def segments(names, pad_cols=None):   # blocks of rows stacked with every block's start at a multiple of 8 rows
             parts = []
@@ -123,6 +145,10 @@ class SeqWeights:
                 w["norm1b"] = norm_w(p + "norm1b")
                 if L.ff or L.moe:
                     w["norm2b"] = norm_w(p + "norm2b")
+            if cfg.layer_scale:
+                for q in ("ls1", "ls2") if (L.ff or L.moe) else ("ls1",):
+                    check(p + q, (W,))
+                    w[q] = f32(get(p + q))
             if hc:
                 n = cfg.streams
                 for q in ("hc1", "hc2") if (L.ff or L.moe) else ("hc1",):
@@ -179,9 +205,12 @@ class SeqWeights:
                     rows.append(m + "dkv")
                     w["a_latent_norm"] = f32(get(m + "dkv.norm"))
                 if a.gate:
-                    check(m + "g", (a.heads, W))
+                    check(m + "g", (a.gate_rows, W))
                     rows.append(m + "g")
-                w["a_in"] = mat(*rows)
+                if a.gate and a.gate_channel:        # the gate block starts at a multiple of 8 rows
+                    w["a_in"] = torch.cat([mat(*rows[:-1]), mat(rows[-1])], 0).contiguous()
+                else:
+                    w["a_in"] = mat(*rows)
                 # query absorption reads each head's key up-projection transposed: [heads][rank][dim]
                 w["a_uk_t"] = get(m + "uk").to(torch.float32).reshape(a.heads, a.dim, a.kv_rank).transpose(1, 2) \
                     .contiguous().to(device=device, dtype=dtype)
@@ -193,15 +222,21 @@ class SeqWeights:
                 w["rot_freq"], w["rot_mag"] = rotary(a.rot)
             elif L.type == "attention":
                 a, m = L.attn, p + "mix."
-                check(m + "q", (a.heads * a.maps * a.dim, W)), check(m + "k", (a.kv_heads * a.maps * a.dim, W)), check(m + "o", (W, a.heads * a.vdim))
+                own_kv = a.kv_from < 0
+                check(m + "q", (a.heads * a.maps * a.dim, W)), check(m + "o", (W, a.heads * a.vdim))
+                if own_kv:
+                    check(m + "k", (a.kv_heads * a.maps * a.dim, W))
+                if a.rel_max:
+                    w["m_bias"] = f32(distance_bias(get(m + "rel"), a.heads, a.rel_max, m + "rel"))
                 if a.maps > 1:      # the second map's weight: one number for the layer
                     dot = lambda u, v: (get(m + u).to(torch.float64) * get(m + v).to(torch.float64)).sum()
                     for n in ("lq1", "lk1", "lq2", "lk2"):
                         check(m + n, (a.dim,))
                     w["m_lambda"] = float(torch.exp(dot("lq1", "lk1")) - torch.exp(dot("lq2", "lk2"))) + a.diff
                 if a.qk_norm and not a.unit_norm:
-                    check(m + "q.norm", (a.dim,)), check(m + "k.norm", (a.dim,))
-                    w["m_qnorm"], w["m_knorm"] = f32(get(m + "q.norm")), f32(get(m + "k.norm"))
+                    for n in ("q", "k") if own_kv else ("q",):
+                        check(m + n + ".norm", (a.dim,))
+                        w[f"m_{n}norm"] = f32(get(m + n + ".norm"))
                 if a.temp:
                     check(m + "temp", (a.heads,))
                     w["m_temp"] = f32(get(m + "temp"))
@@ -211,8 +246,8 @@ class SeqWeights:
                         raise ValueError(f"{m}vmix is not a single number")
                     w["m_vmix_role"] = 1 if first == i else 2
                     w["m_vmix"] = float(get(m + "vmix").to(torch.float32).reshape(-1)[0])
-                rows = [m + "q", m + "k"]
-                if not a.value_keys:
+                rows = [m + "q", m + "k"] if own_kv else [m + "q"]
+                if not a.value_keys and own_kv:
                     check(m + "v", (a.kv_heads * a.vdim, W))
                     rows.append(m + "v")
                 if a.gate != "none":
@@ -279,6 +314,9 @@ class SeqWeights:
                 for j in range(e.experts):
                     check(f"{m}e{j}.up", (e.ff, W)), check(f"{m}e{j}.down", (W, e.ff))
                 check(m + "router", (e.outputs, W))
+                if e.router_bias:
+                    check(m + "router.b", (e.outputs,))
+                    w["e_router_bias"] = f32(get(m + "router.b"))
                 if e.router != "topk_softmax" and e.correction:
                     check(m + "correction", (e.outputs,))
                 if e.act in ("clamp_glu", "silu_glu"):
@@ -293,7 +331,7 @@ class SeqWeights:
                         g, u = get(f"{m}e{j}.gate"), get(f"{m}e{j}.up")
                         if not w["e_up_il16"]:
                             return torch.cat([g, u], 0)
-                        return torch.stack([g.view(e.ff // 16, 16, W), u.view(e.ff // 16, 16, W)], 1).reshape(2 * e.ff, W)
+                        return il16(g, u)
 
                     w["e_up"] = torch.stack([gate_up(j) for j in range(e.experts)]).to(device=device, dtype=dtype).contiguous()
                 else:
@@ -317,7 +355,11 @@ class SeqWeights:
                     w["ff_in"] = mat(p + "mlp.up")
                 else:
                     check(p + "mlp.gate", (L.ff, W))
-                    w["ff_in"] = mat(p + "mlp.gate", p + "mlp.up")
+                    w["ff_il16"] = int(cfg.dense == "clamp_glu" and L.ff % 16 == 0)
+                    if w["ff_il16"]:
+                        w["ff_in"] = il16(get(p + "mlp.gate"), get(p + "mlp.up")).to(device=device, dtype=dtype).contiguous()
+                    else:
+                        w["ff_in"] = mat(p + "mlp.gate", p + "mlp.up")
                 w["ff_out"] = mat(p + "mlp.down")
             self.layers.append(w)
         for i, L in enumerate(cfg.layers):
@@ -329,6 +371,12 @@ class SeqWeights:
         n = sum(x.numel() * x.element_size() for x in {id(x): x for x in (self.embed, self.head, self.final_norm)}.values())
         own = {id(w): w for w in self.layers}.values()      # layers that share tensors count once
         return n + sum(x.numel() * x.element_size() for w in own for x in w.values() if isinstance(x, torch.Tensor))
+
+
+def shared_mask(cfg: SeqModelConfig, i: int) -> Tuple[int, int]:
+    """(window, kept first positions) of the pages of attention layer i: what it and every layer that reads its pages still see."""
+    users = [L.attn for j, L in enumerate(cfg.layers) if L.type == "attention" and (j == i or L.attn.kv_from == i)]
+    return (max(a.window for a in users) if all(a.window for a in users) else 0), max(a.keep_first for a in users)
 
 
 class SeqLMForCausalLM:
@@ -344,12 +392,14 @@ class SeqLMForCausalLM:
         self._native = self._build_native()
         attn = {i: (L.left.kv_heads, L.left.dim, L.left.vdim, L.left.chunk) for i, L in enumerate(config.layers) if L.type == "parallel"}
         # sliding-window attention: (kv heads, key size (both maps of a differential head), value size, no chunks, window, kept first positions)
-        attn.update({i: (L.attn.kv_heads, L.attn.maps * L.attn.dim, L.attn.vdim, 0, L.attn.window, L.attn.keep_first) for i, L in enumerate(config.layers) if L.type == "attention"})
+        attn.update({i: (L.attn.kv_heads, L.attn.maps * L.attn.dim, L.attn.vdim, 0) + shared_mask(config, i)
+                     for i, L in enumerate(config.layers) if L.type == "attention" and L.attn.kv_from < 0})
         # a latent cache is one K pool of [latent | rotary key part] rows; a layer that reads another layer's cache has none
         attn.update({i: (1, L.latent.kv_rank + L.latent.rot_dim, 0, 0, L.latent.window) for i, L in enumerate(config.layers)
                      if L.type == "latent_attention" and L.latent.kv_from < 0})
         self._kv_source = {i: (L.latent.kv_from if L.latent.kv_from >= 0 else i) for i, L in enumerate(config.layers)
                            if L.type == "latent_attention"}
+        self._kv_source.update({i: L.attn.kv_from for i, L in enumerate(config.layers) if L.type == "attention" and L.attn.kv_from >= 0})
         pages = (max_tokens + PAGE_SIZE - 1) // PAGE_SIZE + 2 if max_tokens else 32
         self.pool = SeqStatePool(attn, self._native.state_floats(), self.dtype, device, initial_pages=pages)
         self._ensure_workspace(max(256, min(max_tokens, 4096)) if max_tokens else 1024, 64)
@@ -387,7 +437,8 @@ class SeqLMForCausalLM:
             e.norm1_bias_f32, e.norm1_alpha = p(lw.get("norm1_bias")), lw.get("norm1_alpha", 0.0)
             e.norm1b_f32, e.norm2b_f32 = p(lw.get("norm1b")), p(lw.get("norm2b"))
             e.hc1_f32, e.hc2_f32 = p(lw.get("hc1")), p(lw.get("hc2"))
-            e.a_kv_from = -1
+            e.ls1_f32, e.ls2_f32 = p(lw.get("ls1")), p(lw.get("ls2"))
+            e.a_kv_from = e.m_kv_from = -1
             e.rot_inv_freq_f32, e.rot_mag = p(lw.get("rot_freq")), lw.get("rot_mag", 1.0)
             e.canon_w_f32 = p(lw.get("canon"))
             if L.type == "channel_delta":
@@ -407,7 +458,8 @@ class SeqLMForCausalLM:
                 e.type = _cabi.MIX_LATENT
                 e.a_heads, e.a_dim, e.a_rot_dim, e.a_vdim, e.a_rank, e.a_kv_from = a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank, a.kv_from
                 e.a_scale = a.scale
-                e.a_q_rank, e.a_window, e.a_gate = a.q_rank, a.window, int(a.gate)
+                e.a_q_rank, e.a_window, e.a_rot_pairs = a.q_rank, a.window, int(a.rot_pairs)
+                e.a_gate = _cabi.GATE_NONE if not a.gate else (_cabi.GATE_CHANNEL if a.gate_channel else _cabi.GATE_HEAD)
                 e.a_uq, e.a_q_norm_f32 = p(lw.get("a_uq")), p(lw.get("a_q_norm"))
                 e.a_in, e.a_latent_norm_f32, e.a_uk_t, e.a_uv = p(lw["a_in"]), p(lw.get("a_latent_norm")), p(lw["a_uk_t"]), p(lw["a_uv"])
                 e.a_sink_f32, e.a_out = p(lw.get("a_sink")), p(lw["a_out"])
@@ -420,6 +472,9 @@ class SeqLMForCausalLM:
                 e.m_scale = a.scale
                 e.m_unit_norm, e.m_vmix_role, e.m_vmix, e.m_temp_f32 = int(a.unit_norm), lw.get("m_vmix_role", 0), lw.get("m_vmix", 0.0), p(lw.get("m_temp"))
                 e.m_no_qk_norm, e.m_keep_first, e.m_maps, e.m_softcap = int(not a.qk_norm), a.keep_first if a.window else 0, a.maps, a.softcap
+                e.m_kv_from, e.m_temp_every, e.m_temp_coef = a.kv_from, a.temp_every, a.temp_coef
+                if "m_bias" in lw:
+                    e.m_bias_f32, e.m_bias_len = p(lw["m_bias"]), lw["m_bias"].shape[1]
                 e.m_lambda, e.m_diff_scale = lw.get("m_lambda", 0.0), 1.0 - a.diff
                 e.m_in_bias_f32, e.m_in_bias = p(lw.get("m_in_bias")), p(lw.get("m_in_bias_st"))
                 e.m_in, e.m_qnorm_f32, e.m_knorm_f32, e.m_out = p(lw["m_in"]), p(lw.get("m_qnorm")), p(lw.get("m_knorm")), p(lw["m_out"])
@@ -449,11 +504,13 @@ class SeqLMForCausalLM:
                 e.e_act = {"clamp_glu": _cabi.EXPERT_CLAMP_GLU, "silu_glu": _cabi.EXPERT_SILU_GLU, "gelu": _cabi.EXPERT_GELU}.get(x.act, _cabi.EXPERT_RELU2)
                 e.e_up_il16, e.e_group_top, e.e_shared_ungated = lw.get("e_up_il16", 0), x.group_top, int(not x.shared_gate)
                 e.norm2_f32, e.e_router, e.e_correction_f32 = p(lw.get("norm2")), p(lw["e_router"]), p(lw.get("e_correction"))
+                e.e_router_bias_f32 = p(lw.get("e_router_bias"))
                 e.e_up, e.e_down = p(lw["e_up"]), p(lw["e_down"])
                 e.e_shared_up, e.e_shared_down = p(lw.get("e_shared_up")), p(lw.get("e_shared_down"))
             elif L.ff:
                 e.ff_kind = _cabi.FF_MLP if cfg.dense == "mlp" else _cabi.FF_GLU
-                e.ff_act = _cabi.ACT_RELU2 if cfg.dense_act == "relu2" else _cabi.ACT_GELU_TANH
+                e.ff_act = _cabi.ACT_CLAMP_GLU if cfg.dense == "clamp_glu" else (_cabi.ACT_RELU2 if cfg.dense_act == "relu2" else _cabi.ACT_GELU_TANH)
+                e.ff_il16, e.ff_limit = lw.get("ff_il16", 0), L.ff_limit
                 e.norm2_f32, e.ff_in, e.ff_out = p(lw.get("norm2")), p(lw["ff_in"]), p(lw["ff_out"])
         desc = _cabi.SeqModelDesc(
             width=cfg.width, vocab=cfg.vocab, n_layers=len(cfg.layers),
@@ -493,9 +550,9 @@ class SeqLMForCausalLM:
         nl = len(self.config.layers)
         pool = self.pool
         st = (C.c_void_p * nl)(*[(pool.state[i][cache.slot].data_ptr() if pool.state[i] is not None else None) for i in range(nl)])
-        src = self._kv_source                       # latent-attention layers: whose K pool they read
+        src = self._kv_source                       # layers that read another layer's pages
         kp = (C.c_void_p * nl)(*[(pool.k[src.get(i, i)].data_ptr() if src.get(i, i) in pool.k else None) for i in range(nl)])
-        vp = (C.c_void_p * nl)(*[(pool.v[i].data_ptr() if pool.v.get(i) is not None else None) for i in range(nl)])
+        vp = (C.c_void_p * nl)(*[(pool.v[src.get(i, i)].data_ptr() if pool.v.get(src.get(i, i)) is not None else None) for i in range(nl)])
         keep += [st, kp, vp]
         return _cabi.SeqEntry(n_new=n_new, past=cache.seq_len, ids=ids_dev.data_ptr(), page_table=cache.page_table.data_ptr(),
                               scalars=cache.scalars.data_ptr() if device_pos else None, layer_state=st, k_pages=kp, v_pages=vp)
