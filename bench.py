@@ -46,7 +46,7 @@ def parse_args():
                          "path (HF bf16 + flash_attention_2, optionally --liger) on the same B200 = the kernel to beat")
     ap.add_argument("--liger", action="store_true", help="hf_gpu: apply_liger_kernel_to_qwen2_vl() first (REF/demo/infer.py:2-3)")
     ap.add_argument("--model", default="7b", choices=["7b", "small"])
-    ap.add_argument("--arch", default="livecc", choices=["livecc", "seq", "kedelorn", "dibedra", "lugizen", "kapitar"],
+    ap.add_argument("--arch", default="livecc", choices=["livecc", "seq", "kedelorn", "dibedra", "lugizen", "kapitar", "poresun"],
                     help="livecc: the streaming video workload (default, the headline metric); seq: prefill / decode throughput of "
                          "the hybrid sequence model (Bimopel) beside the Qwen2-style decoder at equal layer sizes; kedelorn: the "
                          "same for Kedelorn (latent attention, retention, routed experts) beside Bimopel and the Qwen2-style decoder; dibedra: "
@@ -54,9 +54,11 @@ def parse_args():
                          "Qwen2-style decoder; lugizen: the same for Lugizen (delta rule, attention, windowed latent attention, routed "
                          "experts, sublayers normed on their output) beside Kedelorn and the Qwen2-style decoder; kapitar: the same for Kapitar "
                          "(differential attention, lightning attention, routed experts, sublayers normed on either side) beside Dibedra, "
-                         "Kedelorn and the Qwen2-style decoder")
-    ap.add_argument("--seq-sizes", default="", help="--arch seq / kedelorn / dibedra / lugizen / kapitar: comma-separated size names (livecc_b200/seq_bench.py SIZES)")
-    ap.add_argument("--seq-prompt", default="1024,4096", help="--arch seq / kedelorn / dibedra / lugizen / kapitar: prompt lengths")
+                         "Kedelorn and the Qwen2-style decoder; poresun: the same for Poresun (attention with distance biases, latent "
+                         "attention, shared keys and values, routed experts, post-norm blocks) beside Dibedra, Kedelorn, Lugizen and "
+                         "the Qwen2-style decoder")
+    ap.add_argument("--seq-sizes", default="", help="--arch seq / kedelorn / dibedra / lugizen / kapitar / poresun: comma-separated size names (livecc_b200/seq_bench.py SIZES)")
+    ap.add_argument("--seq-prompt", default="1024,4096", help="--arch seq / kedelorn / dibedra / lugizen / kapitar / poresun: prompt lengths")
     ap.add_argument("--seconds", type=int, default=60, help="clip length in seconds of video (2 fps)")
     ap.add_argument("--size", type=int, default=448)
     ap.add_argument("--max-new-tokens", type=int, default=16)
@@ -499,10 +501,10 @@ def run_hf_gpu(args, cfg, config, dev):
 # ------------------------------------------------------------------------------------------------
 def main():
     args = parse_args()
-    if args.arch in ("seq", "kedelorn", "dibedra", "lugizen", "kapitar"):
+    if args.arch in ("seq", "kedelorn", "dibedra", "lugizen", "kapitar", "poresun"):
         from livecc_b200 import seq_bench
 
-        print(json.dumps(seq_bench.main(args, design={"kedelorn": "Kedelorn", "dibedra": "Dibedra", "lugizen": "Lugizen", "kapitar": "Kapitar"}.get(args.arch, "Bimopel"))), flush=True)
+        print(json.dumps(seq_bench.main(args, design={"kedelorn": "Kedelorn", "dibedra": "Dibedra", "lugizen": "Lugizen", "kapitar": "Kapitar", "poresun": "Poresun"}.get(args.arch, "Bimopel"))), flush=True)
         return
     from livecc_b200 import runner  # the repo's own multi-GPU plumbing (rank env, NCCL init, barrier + device sync)
 

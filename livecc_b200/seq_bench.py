@@ -129,6 +129,33 @@ def kapitar_config(width: int, n_layers: int, ff: int, window: int, vocab: int =
     return SeqModelConfig.from_json({"architecture": "Kapitar", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": 1e-6}})
 
 
+def poresun_config(width: int, n_layers: int, ff: int, window: int, vocab: int = 32768) -> SeqModelConfig:
+    """Post-norm blocks; layers in the pattern causal attention with a query temperature, sliding-window attention with scores capped
+    at 50, latent attention, causal attention that reads the first one's keys and values. Attention: 128-channel heads, 8 query heads
+    per key/value head, 32 distance buckets up to 1024 positions. Latent attention as in lugizen_config, without a window and with a
+    gate per channel. The first layer has a clamped gated feed-forward of width ff, every other layer 16 two-matrix experts of width
+    ff/4, 4 per token, beside a shared expert of width ff/2: every token reads 3 x width x ff feed-forward weights, the dense gated `ff`
+    of the models beside it."""
+    heads, layers = width // 128, []
+    att = dict(heads=heads, kv_heads=max(1, heads // 8), dim=128, vdim=128, scale=128 ** -0.5, bias_max=1024, bias_rows=32)
+    moe = {"kind": "moe", "expert": {"ff": ff // 4 // 8 * 8}, "router": {"experts": 16, "top": 4}, "shared": {"ff": ff // 2 // 8 * 8}}
+    for i in range(n_layers):
+        k = i % 4
+        if k == 1:
+            L = {"type": "attention", "mixer": dict(att, mask={"size": window}, softcap=50.0)}
+        elif k == 2:
+            L = {"type": "latent_attention", "mixer": dict(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=192, q_rank=3 * width // 8,
+                                                           rot={"dims": 64, "base": 10000.0}, scale=192 ** -0.5)}
+        else:
+            L = {"type": "attention_2", "mixer": dict(att, q_temp={"coef": 0.1, "every": 1024})}
+            if k == 3:
+                L["mixer"]["kv_from"] = i - 3
+        L["mlp"] = {"kind": "dense", "ff": ff // 16 * 16, "limit": 7.0} if i == 0 else moe
+        layers.append(L)
+    return SeqModelConfig.from_json({"architecture": "Poresun", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": 1e-6},
+                                     "postln_alpha": 2.0, "embedding": {"scale": 1.0}})
+
+
 def qwen_config(width: int, n_layers: int, ff: int, vocab: int = 32768) -> LiveCCConfig:
     heads = width // 128
     return LiveCCConfig(
@@ -199,10 +226,11 @@ def run(sizes: List[str], prompt_lens: List[int], new_tokens: int, steps: int, w
         width, n_layers, ff, chunk = SIZES[name]
         rec = {}
         arms = {"Bimopel": ["bimopel"], "Kedelorn": ["kedelorn", "bimopel"], "Dibedra": ["dibedra", "kedelorn"],
-                "Lugizen": ["lugizen", "kedelorn"], "Kapitar": ["kapitar", "dibedra", "kedelorn"]}[design]
+                "Lugizen": ["lugizen", "kedelorn"], "Kapitar": ["kapitar", "dibedra", "kedelorn"],
+                "Poresun": ["poresun", "dibedra", "kedelorn", "lugizen"]}[design]
         make = {"bimopel": lambda: seq_config(width, n_layers, ff, chunk), "kedelorn": lambda: kedelorn_config(width, n_layers, ff),
                 "dibedra": lambda: dibedra_config(width, n_layers, ff, chunk), "lugizen": lambda: lugizen_config(width, n_layers, ff, chunk),
-                "kapitar": lambda: kapitar_config(width, n_layers, ff, chunk)}
+                "kapitar": lambda: kapitar_config(width, n_layers, ff, chunk), "poresun": lambda: poresun_config(width, n_layers, ff, chunk)}
         for label, cfg in [(a, make[a]()) for a in arms]:
             m = SeqLMForCausalLM.from_state_dict(cfg, synthetic_seq_tensors(cfg, seed=7, device="cuda"), dtype,
                                                  max_tokens=max(prompt_lens) + new_tokens + 64)
@@ -225,7 +253,7 @@ def run(sizes: List[str], prompt_lens: List[int], new_tokens: int, steps: int, w
 
 
 def main(args, design: str = "Bimopel") -> Dict:
-    """bench.py --arch seq | kedelorn | dibedra | lugizen | kapitar: one JSON line; `value` = decode tokens/s of the first size at the first prompt length."""
+    """bench.py --arch seq | kedelorn | dibedra | lugizen | kapitar | poresun: one JSON line; `value` = decode tokens/s of the first size at the first prompt length."""
     sizes = [s for s in (args.seq_sizes.split(",") if args.seq_sizes else list(SIZES)) if s in SIZES]
     lens = [int(x) for x in args.seq_prompt.split(",")]
     res = run(sizes, lens, args.max_new_tokens if args.max_new_tokens > 16 else 64, args.steps, max(args.warmup, 3), design=design)
@@ -233,7 +261,8 @@ def main(args, design: str = "Bimopel") -> Dict:
     return {"metric": "decode_tokens_per_s", "value": first["decode_tok_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
             "warmup": max(args.warmup, 3), "ms_per_step": first["decode_ms_per_token"], "higher_is_better": True, "dtype": "bf16",
             "data": "synthetic (random weights, random ids)", "vs_baseline": None,
-            "config": {"model": f"{design} {sizes[0]} beside " + {"Kedelorn": "Bimopel and the ", "Dibedra": "Kedelorn and the ", "Lugizen": "Kedelorn and the ", "Kapitar": "Dibedra, Kedelorn and the "}.get(design, "") +
+            "config": {"model": f"{design} {sizes[0]} beside " + {"Kedelorn": "Bimopel and the ", "Dibedra": "Kedelorn and the ", "Lugizen": "Kedelorn and the ", "Kapitar": "Dibedra, Kedelorn and the ",
+                                                                           "Poresun": "Dibedra, Kedelorn, Lugizen and the "}.get(design, "") +
                                 "Qwen2-style decoder of equal width/depth/ff", "global_batch": 1,
                        "seq_len": lens[0], "parallelism": "1 gpu", "l2": "weights of every size exceed L2"},
             "sizes": res}
