@@ -1,5 +1,5 @@
 """Hybrid sequence models (decoder-only language models built from state-space, gated-linear-attention, delta-rule, chunk-local
-attention, retention, lightning, latent-attention, sliding-window and differential attention mixers, in post-norm blocks, pre-norm
+attention, retention, lightning, latent-attention, sliding-window, distance-biased and differential attention mixers, in post-norm blocks, pre-norm
 blocks on several residual streams, parallel blocks, blocks normed on the sublayer's output or on either side of it, with dense or
 routed feed-forwards) behind the same surface as the video-language engine: `from_pretrained`, `generate`, a cache object that callers pass back, greedy token selection in the library's sampling kernel.
 
